@@ -35,12 +35,13 @@ from ..native import HostCore
 @dataclasses.dataclass(frozen=True)
 class GroupSpec:
     """A cache group: which tokens its layers read (``window`` None = all; ``chunk`` C: from the start of the
-    query's own run of C positions on) and its pool."""
+    query's own run of C positions on; ``keep_first`` K: the first K tokens as well) and its pool."""
     key: Tuple
     window: Optional[int]
     page_size: int
     num_pages: int
     chunk: Optional[int] = None
+    keep_first: int = 0
 
     @property
     def keeps_all(self) -> bool:
@@ -162,7 +163,7 @@ class CacheManager:
         if max_context is None:
             max_context = max([g.num_pages * g.page_size for g in self.groups if g.keeps_all] or
                               [g.num_pages * g.page_size for g in self.groups] or [1])
-        self.core = HostCore([(g.window, g.page_size, g.num_pages, g.chunk) for g in self.groups], max_requests,
+        self.core = HostCore([(g.window, g.page_size, g.num_pages, g.chunk, g.keep_first) for g in self.groups], max_requests,
                              max_tokens_per_step or max(max_requests, 1), max(1, max_context))
         self._names = _Names()
         self.pools = [PagePool(g.num_pages, self.core, i, self._names) for i, g in enumerate(self.groups)]
@@ -193,7 +194,8 @@ class CacheManager:
 
     # -- page arithmetic -----------------------------------------------------------
     def first_needed_page(self, g: int, ctx_len: int) -> int:
-        """Logical index of the first page a query at position >= ctx_len can still read."""
+        """Logical index of the first page a query at position >= ctx_len can still read (the pages of kept first
+        tokens aside, see ``GroupSpec.keep_first``)."""
         spec = self.groups[g]
         first_key = 0
         if spec.window is not None:

@@ -57,6 +57,10 @@ def _builtin():
         from .gevovik import GevovikConfig
         register_architecture("Gevovik", GevovikConfig.from_json, gevovik.build_plan,
                               complete_config=lambda cfg, shapes: cfg.with_shapes(shapes))
+    if "Duzizen" not in _REGISTRY:
+        from ..architectures import duzizen
+        from .duzizen import DuzizenConfig
+        register_architecture("Duzizen", DuzizenConfig.from_json, duzizen.build_plan)
     if "Dufizen" not in _REGISTRY:
         from ..architectures import dufizen
         from .dufizen import DufizenConfig

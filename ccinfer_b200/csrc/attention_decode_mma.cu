@@ -75,7 +75,8 @@ attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     const int* bt = block_table + (size_t)b * bt_stride;
     const int page_shift = (page_size & (page_size - 1)) == 0 ? 31 - __clz(page_size) : -1;
     const int j0 = first_visible_key(p, window, ex.chunk);
-    const int first_tile = j0 / kTileKeys, last_tile = p / kTileKeys;
+    const KeyTiles kt(j0, ex.keep, kTileKeys);
+    const int first_tile = kt.first, last_tile = p / kTileKeys;
     const int n_tiles = last_tile - first_tile + 1;
     const int per_split = (n_tiles + num_splits - 1) / num_splits;
     const int my_first = first_tile + split * per_split;
@@ -88,8 +89,8 @@ attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     auto issue = [&](int tile, int stage) {
       __nv_bfloat16* ks_ = k_s + stage * TILE_ELEMS;
       __nv_bfloat16* vs_ = v_s + stage * TILE_ELEMS;
-      const int j = tile * kTileKeys + ld_row;
-      bool valid = j >= j0 && j <= p;
+      const int j = kt.tile(tile) * kTileKeys + ld_row;
+      bool valid = key_visible(j, j0, p, ex.keep);
       size_t src = 0;
       if (valid) {
         const int lp = page_shift >= 0 ? (j >> page_shift) : (j / page_size);
@@ -141,14 +142,14 @@ attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
         }
       }
       // mask, online softmax (rows gid and gid + 8)
-      const int jbase = (my_first + it) * kTileKeys + warp * 16 + 2 * tig;
+      const int jbase = kt.tile(my_first + it) * kTileKeys + warp * 16 + 2 * tig;
       float mx0 = -CUDART_INF_F, mx1 = -CUDART_INF_F;
 #pragma unroll
       for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int j = jbase + nb * 8 + e;
-          const bool vis = j >= j0 && j <= p;
+          const bool vis = key_visible(j, j0, p, ex.keep);
           s[nb][e] = vis ? s[nb][e] * scale : -CUDART_INF_F;
           s[nb][2 + e] = vis ? s[nb][2 + e] * scale : -CUDART_INF_F;
           mx0 = fmaxf(mx0, s[nb][e]);
@@ -314,12 +315,12 @@ CCB_API int ccb_attention_decode_mma(const void* q, const void* k_cache, const v
                                      float* part_acc, float* part_ml, const int* positions,
                                      const int* entry_of_token, const int* block_table, int bt_stride,
                                      int n_entries, int row0, int n_rows, int nq, int nkv, int hd, int page_size,
-                                     int num_pages, int window, float scale, int num_splits, int chunk,
+                                     int num_pages, int window, float scale, int num_splits, int chunk, int keep,
                                      const float* sink, const void* gate, int gate_stride, int* status,
                                      cudaStream_t stream) {
   if (n_rows <= 0) return 0;
-  if (chunk < 0 || (gate != nullptr && gate_stride < nq)) return CCB_REFUSE_ARG;
-  const AttnExtra ex{chunk, sink, gate, gate_stride};
+  if (chunk < 0 || keep < 0 || (gate != nullptr && gate_stride < nq)) return CCB_REFUSE_ARG;
+  const AttnExtra ex{chunk, sink, gate, gate_stride, keep};
   if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || page_size <= 0 || bt_stride <= 0 || num_splits <= 0 ||
       num_splits > 64)
     return CCB_REFUSE_SIZE;

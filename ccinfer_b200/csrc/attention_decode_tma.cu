@@ -111,7 +111,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
   // merges, they leave at once and are not waited for (measured at one row and 2,048 keys with a grid of
   // 32 splits: 12.1 us when all 32 took a tile and were merged, as against 10.6 us with a grid of 8).
   const int j0 = padded ? 0 : first_visible_key(p, window, ex.chunk);
-  const int first_tile = j0 / kTileKeys, last_tile = (padded ? 0 : p) / kTileKeys;
+  const KeyTiles kt(j0, ex.keep, kTileKeys);
+  const int first_tile = kt.first, last_tile = (padded ? 0 : p) / kTileKeys;
   const int n_tiles = last_tile - first_tile + 1;
   const int eff_splits = padded ? 1 : min(num_splits, max(1, (n_tiles + kMinSplitTiles - 1) / kMinSplitTiles));
   if (counters != nullptr && split >= eff_splits) return;
@@ -235,14 +236,14 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
       if (lane == 0) mbar_expect_tx(bar0 + 8 * stage, TILE_BYTES);
       __syncwarp();
       if (lane < pages_per_tile) {
-        const int lp = ((tile * kTileKeys) >> page_shift) + lane;
+        const int lp = ((kt.tile(tile) * kTileKeys) >> page_shift) + lane;
         int page = (lp <= lp_last && lp < bt_stride) ? bt[lp] : -1;
         if (page < 0 || page >= num_pages) {
           // A page the tile reaches but no query of the row reads (before the window, beyond the position)
           // is replaced by one that certainly exists and its keys are masked.  One that holds a visible key
           // must be there: its absence is reported, not papered over.
           const int k_lo = lp << page_shift;
-          if (k_lo <= p_seen && k_lo + page_size - 1 >= j0) set_status(status, CCB_ST_BAD_PAGE);
+          if (k_lo <= p_seen && (k_lo + page_size - 1 >= j0 || k_lo < ex.keep)) set_status(status, CCB_ST_BAD_PAGE);
           page = bt[lp_last];
         }
         if (page < 0 || page >= num_pages) {
@@ -299,14 +300,14 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
         }
       }
       // mask, online softmax (rows gid and gid + 8)
-      const int jbase = (my_first + it) * kTileKeys + warp * 16 + 2 * tig;
+      const int jbase = kt.tile(my_first + it) * kTileKeys + warp * 16 + 2 * tig;
       float mx0 = -CUDART_INF_F, mx1 = -CUDART_INF_F;
 #pragma unroll
       for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int j = jbase + nb * 8 + e;
-          const bool vis = j >= j0 && j <= p_seen;
+          const bool vis = key_visible(j, j0, p_seen, ex.keep);
           s[nb][e] = vis ? s[nb][e] * scale : -CUDART_INF_F;
           s[nb][2 + e] = vis ? s[nb][2 + e] * scale : -CUDART_INF_F;
           mx0 = fmaxf(mx0, s[nb][e]);
@@ -611,7 +612,7 @@ int launch(const void* q, const FusedQkv& fq, const void* k_cache, const void* v
 }  // namespace
 
 // As ccb_attention_decode_mma, for page sizes that are a power of two from 8 to 64 (others: CCB_REFUSE_SIZE).
-// chunk, sink, gate, gate_stride: see AttnExtra (0 / null: none).
+// chunk, keep, sink, gate, gate_stride: see AttnExtra (0 / null: none).
 // `counters` (optional): n_rows * kv_heads * ceil(group / 16) ints that are zero before the first launch and
 // are left zero; with them the splits are merged by the attention kernel itself, without them by a second
 // kernel.
@@ -620,11 +621,11 @@ CCB_API int ccb_attention_decode_tma(const void* q, const void* k_cache, const v
                                      const int* entry_of_token, const int* block_table, int bt_stride,
                                      int n_entries, int row0, int n_rows, int nq, int nkv, int hd, int page_size,
                                      int num_pages, int window, float scale, int num_splits, int* counters,
-                                     int chunk, const float* sink, const void* gate, int gate_stride,
+                                     int chunk, int keep, const float* sink, const void* gate, int gate_stride,
                                      int* status, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
-  if (chunk < 0 || (gate != nullptr && gate_stride < nq)) return CCB_REFUSE_ARG;
-  const AttnExtra ex{chunk, sink, gate, gate_stride};
+  if (chunk < 0 || keep < 0 || (gate != nullptr && gate_stride < nq)) return CCB_REFUSE_ARG;
+  const AttnExtra ex{chunk, sink, gate, gate_stride, keep};
   if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || bt_stride <= 0 || num_splits <= 0 || num_splits > 64 ||
       page_size < 8 || page_size > 64 || (page_size & (page_size - 1)) != 0 ||
       ((reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & 15) != 0)
@@ -657,11 +658,11 @@ CCB_API int ccb_attention_decode_tma_fused(const void* qkv, int qkv_stride, void
                                            int page_size, int num_pages, int window, float scale, int num_splits,
                                            const float* q_w, const float* k_w, float eps, const float* inv_freq,
                                            int write_kv, const float* bias, float qt_coef, int qt_every,
-                                           int* counters, int chunk, const float* sink, const void* gate,
+                                           int* counters, int chunk, int keep, const float* sink, const void* gate,
                                            int gate_stride, int* status, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
-  if (chunk < 0 || (gate != nullptr && gate_stride < nq)) return CCB_REFUSE_ARG;
-  const AttnExtra ex{chunk, sink, gate, gate_stride};
+  if (chunk < 0 || keep < 0 || (gate != nullptr && gate_stride < nq)) return CCB_REFUSE_ARG;
+  const AttnExtra ex{chunk, sink, gate, gate_stride, keep};
   if (qt_every < 0 || (bias != nullptr && !write_kv)) return CCB_REFUSE_ARG;
   if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || bt_stride <= 0 || num_splits <= 0 || num_splits > 64 ||
       page_size < 8 || page_size > 64 || (page_size & (page_size - 1)) != 0 || (qkv_stride & 1) ||

@@ -72,7 +72,8 @@ attention_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
   cp_async_commit();
 
   const int j_lo = first_visible_key(p_first, window, ex.chunk);  // first key any row sees
-  const int first_tile = j_lo / kKTile, last_tile = p_last / kKTile;
+  const KeyTiles kt(j_lo, ex.keep, kKTile);
+  const int first_tile = kt.first, last_tile = p_last / kKTile;
   const int n_tiles = last_tile - first_tile + 1;
 
   // Two threads share a key row: one page lookup and one address per thread and tile, then 16-byte copies of
@@ -82,8 +83,8 @@ attention_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
   auto issue = [&](int tile, int stage) {
     __nv_bfloat16* ks_ = k_s + stage * TILE_ELEMS;
     __nv_bfloat16* vs_ = v_s + stage * TILE_ELEMS;
-    const int j = tile * kKTile + ld_row;
-    bool valid = j >= j_lo && j <= p_last;
+    const int j = kt.tile(tile) * kKTile + ld_row;
+    bool valid = key_visible(j, j_lo, p_last, ex.keep);
     size_t src = 0;
     if (valid) {
       const int lp = page_shift >= 0 ? (j >> page_shift) : (j / page_size);
@@ -140,9 +141,9 @@ attention_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
     cp_async_commit();
     const __nv_bfloat16* ks_ = k_s + (it % kPStages) * TILE_ELEMS;
     const __nv_bfloat16* vs_ = v_s + (it % kPStages) * TILE_ELEMS;
-    const int jt = (first_tile + it) * kKTile;
+    const int jt = kt.tile(first_tile + it) * kKTile;
     // a warp whose rows all lie before this tile's first key has nothing to do in it (causal)
-    const bool warp_active = jt <= p_first + warp * 16 + 15 && jt + kKTile > warp_lo;
+    const bool warp_active = jt <= p_first + warp * 16 + 15 && (jt + kKTile > warp_lo || jt < ex.keep);
     if (warp_active) {
       float s[8][4];
 #pragma unroll
@@ -167,8 +168,8 @@ attention_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfl
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int j = jt + nb * 8 + 2 * tig + e;
-          s[nb][e] = (j <= pr0 && j >= lo0) ? s[nb][e] * scale_log2 : -CUDART_INF_F;
-          s[nb][2 + e] = (j <= pr1 && j >= lo1) ? s[nb][2 + e] * scale_log2 : -CUDART_INF_F;
+          s[nb][e] = key_visible(j, lo0, pr0, ex.keep) ? s[nb][e] * scale_log2 : -CUDART_INF_F;
+          s[nb][2 + e] = key_visible(j, lo1, pr1, ex.keep) ? s[nb][2 + e] * scale_log2 : -CUDART_INF_F;
           mx0 = fmaxf(mx0, s[nb][e]);
           mx1 = fmaxf(mx1, s[nb][2 + e]);
         }
@@ -277,20 +278,20 @@ int launch(const void* q, const void* k_cache, const void* v_cache, void* out, c
 
 // Requests entry0 .. entry0 + n_entries - 1 of the step (cu_q, pos0 and block_table rows are indexed by the
 // request's place in the step); max_new = the most new tokens any of them brings.  bfloat16, head size 64
-// or 128; other sizes are refused and belong to ccb_attention_split.  chunk, sink, gate, gate_stride: see AttnExtra
+// or 128; other sizes are refused and belong to ccb_attention_split.  chunk, keep, sink, gate, gate_stride: see AttnExtra
 // (0 / null: none).
 CCB_API int ccb_attention_prefill_mma(const void* q, const void* k_cache, const void* v_cache, void* out,
                                       const int* cu_q, const int* pos0, const int* block_table, int bt_stride,
                                       int entry0, int n_entries, int max_new, int nq, int nkv, int hd,
-                                      int page_size, int num_pages, int window, float scale, int chunk,
+                                      int page_size, int num_pages, int window, float scale, int chunk, int keep,
                                       const float* sink, const void* gate, int gate_stride, int* status,
                                       cudaStream_t stream) {
   if (n_entries <= 0 || max_new <= 0) return 0;
   if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || page_size <= 0 || bt_stride <= 0 || n_entries > 65535 || nq > 65535 ||
-      chunk < 0)
+      chunk < 0 || keep < 0)
     return CCB_REFUSE_SIZE;
   if (gate != nullptr && gate_stride < nq) return CCB_REFUSE_ARG;
-  const AttnExtra ex{chunk, sink, gate, gate_stride};
+  const AttnExtra ex{chunk, sink, gate, gate_stride, keep};
   if (hd == 128)
     return launch<128>(q, k_cache, v_cache, out, cu_q, pos0, block_table, bt_stride, entry0, n_entries, max_new,
                        nq, nkv, page_size, num_pages, window, scale, ex, status, stream);

@@ -119,7 +119,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
   const int p_first = p0 + q_first, p_last = p_first + rows_here - 1;
   const int* bt = block_table + (size_t)b * bt_stride;
   const int j_lo = first_visible_key(p_first, window, ex.chunk);   // the first key any row of the tile sees
-  const int first_tile = j_lo / kTK, last_tile = p_last / kTK;
+  const KeyTiles kt(j_lo, ex.keep, kTK);
+  const int first_tile = kt.first, last_tile = p_last / kTK;
   const int n_tiles = last_tile - first_tile + 1;
 
   if (threadIdx.x == 0) {
@@ -164,12 +165,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
                                                // reaches but the request does not hold (their keys are masked)
     // first row (in the [rows, HD] view of the cache) of this lane's page of tile t
     auto page_row = [&](int t) -> int {
-      const int lp = (((first_tile + t) * kTK) >> page_shift) + lane;
+      const int lp = ((kt.tile(first_tile + t) * kTK) >> page_shift) + lane;
       int page = (lp <= lp_last && lp < bt_stride) ? bt[lp] : -1;
       if (page < 0 || page >= num_pages) {
         // stands in only for pages none of the tile's queries reads; a missing page with a visible key is reported
         const int k_lo = lp << page_shift;
-        if (k_lo <= p_last && k_lo + page_size - 1 >= j_lo) set_status(status, CCB_ST_BAD_PAGE);
+        if (k_lo <= p_last && (k_lo + page_size - 1 >= j_lo || k_lo < ex.keep)) set_status(status, CCB_ST_BAD_PAGE);
         page = bt[lp_last];
       }
       if (page < 0 || page >= num_pages) {
@@ -265,7 +266,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
       alive = mbar_wait(b_sf + 8 * (i & 1), (i >> 1) & 1);
       if (!alive) break;
       tc_fence_after();
-      const int jt = (first_tile + i) * kTK;
+      const int jt = kt.tile(first_tile + i) * kTK;
       const uint32_t tmem_si = tmem_s + (i & 1) * 128;
       // Most tiles lie wholly in every row's past (and inside its window): they need no mask.
       const bool need_mask = (jt + kTK - 1 > p_first) || jt < lo_last;
@@ -278,7 +279,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
 #pragma unroll
         for (int e = 0; e < kTK; ++e) {
           const int j = jt + e;
-          if (!(j <= pr && j >= lo)) v[e] = 0xff800000u;  // -inf: 2^(-inf) = 0 below
+          if (!key_visible(j, lo, pr, ex.keep)) v[e] = 0xff800000u;  // -inf: 2^(-inf) = 0 below
         }
       }
       float mx4[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};  // four independent chains
@@ -442,7 +443,8 @@ attention_prefill_tc_pair_kernel(const __grid_constant__ CUtensorMap tmQ, const 
   const int p_first = p0 + q_first, p_last = p_first + rows_here - 1;
   const int* bt = block_table + (size_t)b * bt_stride;
   const int j_lo = first_visible_key(p_first, window, ex.chunk);   // the first key any row of the tile sees
-  const int first_tile = j_lo / kTK, last_tile = p_last / kTK;
+  const KeyTiles kt(j_lo, ex.keep, kTK);
+  const int first_tile = kt.first, last_tile = p_last / kTK;
   const int n_tiles = last_tile - first_tile + 1;
 
   if (threadIdx.x == 0) {
@@ -485,11 +487,11 @@ attention_prefill_tc_pair_kernel(const __grid_constant__ CUtensorMap tmQ, const 
     const int pages_per_tile = kTK >> page_shift;
     const int lp_last = p_last >> page_shift;
     auto page_row = [&](int t) -> int {
-      const int lp = (((first_tile + t) * kTK) >> page_shift) + lane;
+      const int lp = ((kt.tile(first_tile + t) * kTK) >> page_shift) + lane;
       int page = (lp <= lp_last && lp < bt_stride) ? bt[lp] : -1;
       if (page < 0 || page >= num_pages) {
         const int k_lo = lp << page_shift;
-        if (k_lo <= p_last && k_lo + page_size - 1 >= j_lo) set_status(status, CCB_ST_BAD_PAGE);
+        if (k_lo <= p_last && (k_lo + page_size - 1 >= j_lo || k_lo < ex.keep)) set_status(status, CCB_ST_BAD_PAGE);
         page = bt[lp_last];
       }
       if (page < 0 || page >= num_pages) {
@@ -591,7 +593,7 @@ attention_prefill_tc_pair_kernel(const __grid_constant__ CUtensorMap tmQ, const 
       alive = mbar_wait(bar_sf, i & 1);
       if (!alive) break;
       tc_fence_after();
-      const int jt = (first_tile + i) * kTK;
+      const int jt = kt.tile(first_tile + i) * kTK;
       const bool need_mask = (jt + kTK - 1 > p_first) || jt < lo_last;
       uint32_t v[kTK];
 #pragma unroll
@@ -601,7 +603,7 @@ attention_prefill_tc_pair_kernel(const __grid_constant__ CUtensorMap tmQ, const 
 #pragma unroll
         for (int e = 0; e < kTK; ++e) {
           const int j = jt + e;
-          if (!(j <= pr && j >= lo)) v[e] = 0xff800000u;
+          if (!key_visible(j, lo, pr, ex.keep)) v[e] = 0xff800000u;
         }
       }
       float mx4[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};  // four chains, two scores a step
@@ -754,17 +756,17 @@ int launch(const void* q, const void* k_cache, const void* v_cache, void* out, c
 }  // namespace
 
 // As ccb_attention_prefill_mma; n_tokens = rows of q / out.  bfloat16, head size 64 or 128, page size a power
-// of two from 8 to 128; anything else is refused (CCB_REFUSE_SIZE) and belongs to the other kernels.  chunk, sink,
-// gate, gate_stride: see AttnExtra (0 / null: none).
+// of two from 8 to 128; anything else is refused (CCB_REFUSE_SIZE) and belongs to the other kernels.  chunk, keep,
+// sink, gate, gate_stride: see AttnExtra (0 / null: none).
 CCB_API int ccb_attention_prefill_tc(const void* q, const void* k_cache, const void* v_cache, void* out,
                                      const int* cu_q, const int* pos0, const int* block_table, int bt_stride,
                                      int entry0, int n_entries, int max_new, int n_tokens, int nq, int nkv, int hd,
-                                     int page_size, int num_pages, int window, float scale, int chunk,
+                                     int page_size, int num_pages, int window, float scale, int chunk, int keep,
                                      const float* sink, const void* gate, int gate_stride, int* status,
                                      cudaStream_t stream) {
   if (n_entries <= 0 || max_new <= 0) return 0;
-  if (chunk < 0 || (gate != nullptr && gate_stride < nq)) return CCB_REFUSE_ARG;
-  const AttnExtra ex{chunk, sink, gate, gate_stride};
+  if (chunk < 0 || keep < 0 || (gate != nullptr && gate_stride < nq)) return CCB_REFUSE_ARG;
+  const AttnExtra ex{chunk, sink, gate, gate_stride, keep};
   if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || bt_stride <= 0 || n_entries > 65535 || nq > 65535 || page_size < 8 ||
       page_size > 128 || (page_size & (page_size - 1)) != 0 ||
       ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) |

@@ -101,7 +101,8 @@ attention_split_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
       }
     const int* bt = block_table + (size_t)b * bt_stride;
     const int j0 = first_visible_key(p, window, ex.chunk);
-    const int first_tile = j0 >> kTileShift, last_tile = p >> kTileShift;
+    const KeyTiles kt(j0, ex.keep, kTile);
+    const int first_tile = kt.first, last_tile = p >> kTileShift;
     const int n_tiles = last_tile - first_tile + 1;
     const int per_split = (n_tiles + num_splits - 1) / num_splits;
     const int my_first = first_tile + split * per_split;
@@ -114,8 +115,8 @@ attention_split_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
       bool valid[kIt];
 #pragma unroll
       for (int it = 0; it < kIt; ++it) {
-        const int j = tile * kTile + it * 4 + kg;
-        valid[it] = j >= j0 && j <= p;
+        const int j = kt.tile(tile) * kTile + it * 4 + kg;
+        valid[it] = key_visible(j, j0, p, ex.keep);
         rows[it] = 0;
         if (valid[it]) {
           const int lp = j / page_size;
@@ -361,20 +362,20 @@ int pick_gt(int hd, const void* q, const void* k, const void* v, void* out, floa
 
 // Scratch: part_acc holds n_rows * nq * num_splits * hd floats, part_ml n_rows * nq * num_splits * 2
 // (both unused with one split).  Rows row0 .. row0 + n_rows - 1 of q / out / positions are handled.
-// chunk, sink, gate, gate_stride: see AttnExtra (0 / null: none).
+// chunk, keep, sink, gate, gate_stride: see AttnExtra (0 / null: none).
 CCB_API int ccb_attention_split_ex(const void* q, const void* k_cache, const void* v_cache, void* out,
                                    float* part_acc, float* part_ml, const int* positions,
                                    const int* entry_of_token, const int* block_table, int bt_stride, int n_entries,
                                    int row0, int n_rows, int nq, int nkv, int hd, int page_size, int num_pages,
-                                   int window, float scale, int num_splits, int chunk, const float* sink,
+                                   int window, float scale, int num_splits, int chunk, int keep, const float* sink,
                                    const void* gate, int gate_stride, int dtype, int* status, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
   if (hd <= 0 || hd % 8 != 0 || hd > 256 || nq <= 0 || nkv <= 0 || nq % nkv != 0 || page_size <= 0 ||
-      bt_stride <= 0 || num_splits <= 0 || num_splits > 64 || chunk < 0)
+      bt_stride <= 0 || num_splits <= 0 || num_splits > 64 || chunk < 0 || keep < 0)
     return CCB_REFUSE_SIZE;
   if (num_splits > 1 && (part_acc == nullptr || part_ml == nullptr)) return CCB_REFUSE_ARG;
   if (gate != nullptr && gate_stride < nq) return CCB_REFUSE_ARG;
-  const AttnExtra ex{chunk, sink, gate, gate_stride};
+  const AttnExtra ex{chunk, sink, gate, gate_stride, keep};
   if (dtype == CCB_F32)
     return pick_gt<float>(hd, q, k_cache, v_cache, out, part_acc, part_ml, positions, entry_of_token, block_table,
                           bt_stride, n_entries, row0, n_rows, nq, nkv, page_size, num_pages, window, scale,
@@ -393,7 +394,7 @@ CCB_API int ccb_attention_split(const void* q, const void* k_cache, const void* 
                                 int num_splits, int dtype, int* status, cudaStream_t stream) {
   return ccb_attention_split_ex(q, k_cache, v_cache, out, part_acc, part_ml, positions, entry_of_token, block_table,
                                 bt_stride, n_entries, row0, n_rows, nq, nkv, hd, page_size, num_pages, window, scale,
-                                num_splits, 0, nullptr, nullptr, 0, dtype, status, stream);
+                                num_splits, 0, 0, nullptr, nullptr, 0, dtype, status, stream);
 }
 
 // ---------------------------------------------------------------------------------------------

@@ -42,6 +42,7 @@ GROUPS = {
     "base": [
         "elementwise.cu",
         "norm.cu",
+        "norm_chain.cu",
         "rope_kv.cu",
         "gemm_f32.cu",
         "gemm_cublas.cu",
@@ -62,6 +63,8 @@ GROUPS = {
     ],
     "recurrent": [
         "short_conv.cu",
+        "qk_rows.cu",
+        "scalar_memory.cu",
         "delta_rule.cu",
         "linear_attention.cu",
         "ssm.cu",

@@ -100,13 +100,17 @@ __device__ __forceinline__ float row_ssq(const float* row, int n, int lane) {
 }
 
 // The gated activation of a feed-forward, as the epilogue of its gate|up product:
-//   limit <= 0:  silu(g) * u
-//   limit  > 0:  g' = min(g, limit), u' = clamp(u, -limit, limit);  g' * sigmoid(alpha g') * (u' + shift)
+//   gelu = 0, limit <= 0:  silu(g) * u
+//   gelu = 0, limit  > 0:  g' = min(g, limit), u' = clamp(u, -limit, limit);  g' * sigmoid(alpha g') * (u' + shift)
+//   gelu = 1:              gelu(g) * u with the tanh form  0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))), written
+//                          as g * sigmoid(2 sqrt(2 / pi) (g + 0.044715 g^3))
 struct CcbGluAct {
   float limit, alpha, shift;
+  int gelu;
 };
 
 __device__ __forceinline__ float glu_act(const CcbGluAct a, float g, float u) {
+  if (a.gelu) return g / (1.f + __expf(-1.5957691216057308f * g * (1.f + 0.044715f * g * g))) * u;
   if (a.limit > 0.f) {
     g = fminf(g, a.limit);
     u = fminf(fmaxf(u, -a.limit), a.limit);
@@ -115,17 +119,31 @@ __device__ __forceinline__ float glu_act(const CcbGluAct a, float g, float u) {
   return g / (1.f + __expf(-g)) * u;
 }
 
+// The same with the accurate exponential (kernels of their own, the 32-bit path).
+__device__ __forceinline__ float glu_act_exact(const CcbGluAct a, float g, float u) {
+  if (a.gelu) return g / (1.f + expf(-1.5957691216057308f * g * (1.f + 0.044715f * g * g))) * u;
+  if (a.limit > 0.f) {
+    g = fminf(g, a.limit);
+    u = fminf(fmaxf(u, -a.limit), a.limit);
+    return g / (1.f + expf(-a.alpha * g)) * (u + a.shift);
+  }
+  return g / (1.f + expf(-g)) * u;
+}
+
 // What an attention kernel takes beside keys and values (all optional):
 //   chunk  > 0: a query at position p sees only keys from floor(p / chunk) * chunk on (runs of `chunk` positions
 //          counted from the start of the sequence), on top of a window if there is one;
 //   sink   float [q heads]: one more term exp(sink[h]) in the softmax denominator of head h, with no key and no
 //          value, not scaled, counted once per query;
-//   gate   [tokens, gate_stride] in the compute type: head h's result is multiplied by sigmoid(gate[t, h]).
+//   gate   [tokens, gate_stride] in the compute type: head h's result is multiplied by sigmoid(gate[t, h]);
+//   keep   > 0: the first `keep` keys of the sequence are seen by every later query, whatever the window and the
+//          chunk leave out.
 struct AttnExtra {
   int chunk;
   const float* sink;
   const void* gate;
   int gate_stride;
+  int keep;
 };
 
 // The first key position a query at position p sees (both bounds are non-decreasing in p).
@@ -137,6 +155,26 @@ __device__ __forceinline__ int first_visible_key(int p, int window, int chunk) {
   }
   return j0;
 }
+
+// Whether a query at position p whose window (or chunk) starts at key lo sees key j.
+__device__ __forceinline__ bool key_visible(int j, int lo, int p, int keep) {
+  return j <= p && (j >= lo || j < keep);
+}
+
+// The tiles of `tile_keys` keys that a walk over the keys of a query (or of a tile of queries whose first window
+// starts at key j0) visits: those of the keys that are always seen, then those from the window's first one on.
+// They are counted in one run of numbers first .. last (the window's last tile): from `window` on a number is the
+// tile itself, below it the tiles count from 0.  Without kept keys, or where the window reaches them, the two are
+// the same.
+struct KeyTiles {
+  int first, window;
+  __device__ __forceinline__ KeyTiles(int j0, int keep, int tile_keys) {
+    window = j0 / tile_keys;
+    const int kept = (keep + tile_keys - 1) / tile_keys;
+    first = window - (kept < window ? kept : window);
+  }
+  __device__ __forceinline__ int tile(int n) const { return n >= window ? n : n - first; }
+};
 
 // The sink's term folded into a finished softmax of head h (maximum mm, sum ll, natural exponent): ll becomes the
 // whole denominator, and the weighted values are to be multiplied by the factor returned.  A row that saw no key

@@ -602,7 +602,7 @@ CCB_API int ccb_gated_linear_recurrence(const float* qn, const float* kn, const 
 CCB_API int ccb_ssm_recurrence(const float* qn, const float* kn, const float* vv, const float* a, const float* dt,
                                float* state, float* out, const int* cu_q, const int* state_slot, int n_entries,
                                int G, int H, int dk, int dv, cudaStream_t stream) {
-  if (a == nullptr || dt == nullptr) return CCB_REFUSE_ARG;
+  if (a == nullptr) return CCB_REFUSE_ARG;   // (dt null: every step size is one)
   return pick_recurrence<false>(qn, kn, vv, a, dt, state, out, cu_q, state_slot, n_entries, G, H, dk, dv, stream,
                                 true);
 }

@@ -140,12 +140,11 @@ CCB_API int ccb_silu_mul(void* act, const void* gate_up, int T_, int F, int bloc
   return ccb_launch_status();
 }
 
-// Gated activation with clamped inputs:
-//   g = min(gate, limit), u = clamp(up, -limit, limit);  act = g * sigmoid(alpha * g) * (u + up_shift)
+// The other gated activations (ccb::glu_act: clamped inputs with a sigmoid gate of its own slope, or tanh gelu)
 // over the same two layouts of the merged gate|up columns as silu_mul.  Arithmetic in float.
 template <typename T>
-__global__ void clamped_glu_kernel(T* __restrict__ act, const T* __restrict__ gu, int F, int B, size_t total,
-                                   float limit, float alpha, float up_shift) {
+__global__ void gated_act_kernel(T* __restrict__ act, const T* __restrict__ gu, int F, int B, size_t total,
+                                 const CcbGluAct a) {
   ccb::pdl_begin();
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t stride = (size_t)gridDim.x * blockDim.x;
@@ -154,15 +153,13 @@ __global__ void clamped_glu_kernel(T* __restrict__ act, const T* __restrict__ gu
     const int f = (int)(i - t * F);
     const T* row = gu + t * 2 * (size_t)F;
     const int gi = (f / B) * 2 * B + f % B;
-    const float g = fminf(to_f32(row[gi]), limit);
-    const float u = fminf(fmaxf(to_f32(row[gi + B]), -limit), limit);
-    act[i] = from_f32<T>(g / (1.0f + expf(-alpha * g)) * (u + up_shift));
+    act[i] = from_f32<T>(glu_act_exact(a, to_f32(row[gi]), to_f32(row[gi + B])));
   }
 }
 
 // bf16, F and the block multiples of 8: eight elements (16 bytes) per thread and access
-__global__ void clamped_glu_bf16x8_kernel(uint4* __restrict__ act, const uint4* __restrict__ gu, int F8, int B8,
-                                          size_t total8, const CcbGluAct a) {
+__global__ void gated_act_bf16x8_kernel(uint4* __restrict__ act, const uint4* __restrict__ gu, int F8, int B8,
+                                        size_t total8, const CcbGluAct a) {
   ccb::pdl_begin();
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t stride = (size_t)gridDim.x * blockDim.x;
@@ -185,28 +182,29 @@ __global__ void clamped_glu_bf16x8_kernel(uint4* __restrict__ act, const uint4* 
   }
 }
 
-CCB_API int ccb_clamped_glu(void* act, const void* gate_up, int T_, int F, int block, float limit, float alpha,
-                            float up_shift, int dtype, cudaStream_t stream) {
+CCB_API int ccb_gated_act(void* act, const void* gate_up, int T_, int F, int block, float limit, float alpha,
+                          float up_shift, int gelu, int dtype, cudaStream_t stream) {
   if (T_ <= 0) return 0;
   if (F <= 0 || block < 0 || (block > 0 && F % block != 0)) return CCB_REFUSE_SIZE;
+  if (!gelu && !(limit > 0.f)) return CCB_REFUSE_ARG;
+  const CcbGluAct a{limit, alpha, up_shift, gelu};
   const int B = block == 0 ? F : block;
   const size_t total = (size_t)T_ * F;
   const int threads = 256;
-  if (dtype == CCB_BF16 && limit > 0.f && (F % 8) == 0 && (B % 8) == 0 &&
+  if (dtype == CCB_BF16 && (F % 8) == 0 && (B % 8) == 0 &&
       ((reinterpret_cast<uintptr_t>(act) | reinterpret_cast<uintptr_t>(gate_up)) & 15) == 0) {
     const size_t total8 = total / 8;
     const size_t want = (total8 + threads - 1) / threads;
-    ccb_launch(clamped_glu_bf16x8_kernel, (int)(want < 148 * 32 ? want : 148 * 32), threads, 0, stream, (uint4*)act,
-               (const uint4*)gate_up, F / 8, B / 8, total8, CcbGluAct{limit, alpha, up_shift});
+    ccb_launch(gated_act_bf16x8_kernel, (int)(want < 148 * 32 ? want : 148 * 32), threads, 0, stream, (uint4*)act,
+               (const uint4*)gate_up, F / 8, B / 8, total8, a);
     return ccb_launch_status();
   }
   const int blocks = (int)((total + threads - 1) / threads < 148 * 16 ? (total + threads - 1) / threads : 148 * 16);
   if (dtype == CCB_F32)
-    ccb_launch(clamped_glu_kernel<float>, blocks, threads, 0, stream, (float*)act, (const float*)gate_up, F, B, total,
-               limit, alpha, up_shift);
+    ccb_launch(gated_act_kernel<float>, blocks, threads, 0, stream, (float*)act, (const float*)gate_up, F, B, total, a);
   else if (dtype == CCB_BF16)
-    ccb_launch(clamped_glu_kernel<__nv_bfloat16>, blocks, threads, 0, stream, (__nv_bfloat16*)act,
-               (const __nv_bfloat16*)gate_up, F, B, total, limit, alpha, up_shift);
+    ccb_launch(gated_act_kernel<__nv_bfloat16>, blocks, threads, 0, stream, (__nv_bfloat16*)act,
+               (const __nv_bfloat16*)gate_up, F, B, total, a);
   else
     return CCB_REFUSE_DTYPE;
   return ccb_launch_status();

@@ -48,6 +48,7 @@ typedef struct ccinfer_group {
   int num_pages;  /* pages of the pool */
   int chunk;      /* C > 0: a query at position p reads the tokens from floor(p / C) * C on (pages behind the run of
                      the next token are given back); may stand beside a window */
+  int keep_first; /* K > 0: every query reads the first K tokens too (beside a window or a chunk); their pages stay */
 } ccinfer_group;
 
 typedef struct ccinfer_options {

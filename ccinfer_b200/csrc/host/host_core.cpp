@@ -220,6 +220,11 @@ struct ccinfer_engine {
     return first_key / groups[g].page_size;
   }
 
+  // pages at the start of a table that are never given back while the sequence lives
+  int kept_pages(int g) const {
+    return groups[g].keep_first > 0 ? (groups[g].keep_first + groups[g].page_size - 1) / groups[g].page_size : 0;
+  }
+
   void undo(Sequence& s) {
     for (size_t g = 0; g < groups.size(); ++g) {
       const int n = s.taken.empty() ? 0 : s.taken[g];
@@ -262,12 +267,13 @@ struct ccinfer_engine {
       if (groups[g].window <= 0 && groups[g].chunk <= 0) continue;
       auto& t = s.tables[g];
       const int first = std::min(first_needed_page((int)g, s.ctx_len), (int)t.size());
+      const int kept = kept_pages((int)g);
       stale.clear();
-      for (int i = 0; i < first; ++i)
+      for (int i = kept; i < first; ++i)
         if (t[i] >= 0) stale.push_back(t[i]);
       if (stale.empty()) continue;
       pools[g].give_back(s.id, stale.data(), (int)stale.size());   // every later query has passed them
-      for (int i = 0; i < first; ++i) t[i] = -1;
+      for (int i = kept; i < first; ++i) t[i] = -1;
     }
   }
 };

@@ -205,13 +205,14 @@ moe_dense_act_vec_kernel(T* __restrict__ act, int ld, const float* __restrict__ 
 }
 
 // The gated form of the same: the product's row holds all gate columns [E F + shared] and then all up columns;
-// act[t, c] = silu(gate) * up * weight, weight = dense_w[t, c / F] for an expert's columns (exact zeros where it
+// act[t, c] = glu(gate, up) * weight (ccb::glu_act; by default silu(gate) * up), or with w_in glu(gate * weight,
+// up * weight), the weight on the expert's input; weight = dense_w[t, c / F] for an expert's columns (exact zeros where it
 // was not chosen) and sigmoid(shared_gate[t * sg_stride]) for the shared expert's (1 where shared_gate is null).
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_dense_glu_act_kernel(T* __restrict__ act, int lda, const T* __restrict__ gu, int ldg,
                          const float* __restrict__ dense_w, const float* __restrict__ shared_gate, int sg_stride,
-                         int rows, int E, int F, int shared) {
+                         int rows, int E, int F, int shared, const CcbGluAct ga, int w_in) {
   ccb::pdl_begin();
   const int width = E * F + shared;
   const size_t total = (size_t)rows * width;
@@ -223,8 +224,8 @@ moe_dense_glu_act_kernel(T* __restrict__ act, int lda, const T* __restrict__ gu,
     else w = shared_gate ? 1.f / (1.f + expf(-shared_gate[t * sg_stride])) : 1.f;
     float v = 0.f;
     if (w != 0.f) {
-      const float g = to_f32(gu[t * ldg + c]), u = to_f32(gu[t * ldg + width + c]);
-      v = g / (1.f + expf(-g)) * u * w;
+      const float wi = w_in ? w : 1.f, wo = w_in ? 1.f : w;
+      v = glu_act_exact(ga, to_f32(gu[t * ldg + c]) * wi, to_f32(gu[t * ldg + width + c]) * wi) * wo;
     }
     act[t * lda + c] = from_f32<T>(v);
   }
@@ -235,7 +236,7 @@ moe_dense_glu_act_kernel(T* __restrict__ act, int lda, const T* __restrict__ gu,
 __global__ void __launch_bounds__(256)
 moe_dense_glu_act_vec_kernel(__nv_bfloat16* __restrict__ act, int lda, const __nv_bfloat16* __restrict__ gu, int ldg,
                              const float* __restrict__ dense_w, const float* __restrict__ shared_gate, int sg_stride,
-                             int rows, int E, int F, int shared) {
+                             int rows, int E, int F, int shared, const CcbGluAct ga, int w_in) {
   ccb::pdl_begin();
   const int width = E * F + shared;
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
@@ -246,6 +247,7 @@ moe_dense_glu_act_vec_kernel(__nv_bfloat16* __restrict__ act, int lda, const __n
     if (e >= 0) w = dense_w[(size_t)t * E + e];
     else w = shared_gate ? 1.f / (1.f + expf(-shared_gate[(size_t)t * sg_stride])) : 1.f;
     uint4 res = make_uint4(0u, 0u, 0u, 0u);
+    const float wi = w_in ? w : 1.f, wo = w_in ? 1.f : w;
     if (w != 0.f) {
       const uint4 gv = *reinterpret_cast<const uint4*>(gu + (size_t)t * ldg + c);
       const uint4 uv = *reinterpret_cast<const uint4*>(gu + (size_t)t * ldg + width + c);
@@ -255,7 +257,7 @@ moe_dense_glu_act_vec_kernel(__nv_bfloat16* __restrict__ act, int lda, const __n
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const float2 g = __bfloat1622float2(gh[i]), u = __bfloat1622float2(uh[i]);
-        rh[i] = __floats2bfloat162_rn(g.x / (1.f + expf(-g.x)) * u.x * w, g.y / (1.f + expf(-g.y)) * u.y * w);
+        rh[i] = __floats2bfloat162_rn(glu_act_exact(ga, g.x * wi, u.x * wi) * wo, glu_act_exact(ga, g.y * wi, u.y * wi) * wo);
       }
     }
     *reinterpret_cast<uint4*>(act + (size_t)t * lda + c) = res;
@@ -425,7 +427,8 @@ __device__ __forceinline__ uint4 ld16_or_zero(const __nv_bfloat16* p, bool ok) {
 }
 
 // MODE 0: C (compute type) = relu(c)^2 * row_w[row];  MODE 1: C (float) = c;  MODE 2: the matrix's rows are
-// gate and up rows in turn and C (compute type) [*, N / 2] = silu(gate) * up * row_w[row].
+// gate and up rows in turn and C (compute type) [*, N / 2] = glu(gate, up) * row_w[row] (ccb::glu_act), or with w_in
+// glu(gate * row_w[row], up * row_w[row]).
 // A [*, lda]: row src_row[r] (MODE 0) or r itself (src_row null).  W_e = W + e * w_expert_stride, rows at ldw.
 // Few rows an expert (tiles of 16, a decode step): the product is a stream of the chosen experts' matrices, and
 // what counts is bytes in flight.  A block takes 8 columns of a tile; its four warps take a quarter of k each
@@ -437,7 +440,7 @@ moe_grouped_rows16_kernel(const __nv_bfloat16* __restrict__ A, int lda, const in
                           const __nv_bfloat16* __restrict__ W, int ldw, long long w_expert_stride,
                           void* __restrict__ Cout, int ldc, const float* __restrict__ row_w,
                           const int* __restrict__ tile_e, const int* __restrict__ tile_r0,
-                          const int* __restrict__ tile_n, int N, int K) {
+                          const int* __restrict__ tile_n, int N, int K, const CcbGluAct ga, int w_in) {
   ccb::pdl_begin();
   constexpr int DEPTH = 4;
   __shared__ float red[3][32][4];
@@ -513,8 +516,10 @@ moe_grouped_rows16_kernel(const __nv_bfloat16* __restrict__ A, int lda, const in
       if (c0 < N) c[0] = __float2bfloat16_rn(v0);
       if (c0 + 1 < N) c[1] = __float2bfloat16_rn(v1);
     } else if (MODE == 2) {   // columns (2 f, 2 f + 1) are gate f and up f: one number of the gated activation
-      if (c0 + 1 < N)
-        ((__nv_bfloat16*)Cout)[g * ldc + (c0 >> 1)] = __float2bfloat16_rn(v0 / (1.f + __expf(-v0)) * v1 * row_w[g]);
+      if (c0 + 1 < N) {
+        const float wr = row_w[g], wi = w_in ? wr : 1.f, wo = w_in ? 1.f : wr;
+        ((__nv_bfloat16*)Cout)[g * ldc + (c0 >> 1)] = __float2bfloat16_rn(glu_act(ga, v0 * wi, v1 * wi) * wo);
+      }
     } else {
       float* c = (float*)Cout + g * ldc + c0;
       if (c0 < N) c[0] = v0;
@@ -529,7 +534,8 @@ __global__ void __launch_bounds__(128)
 moe_grouped_f32_kernel(const float* __restrict__ A, int lda, const int* __restrict__ src_row,
                        const float* __restrict__ W, int ldw, long long w_expert_stride, float* __restrict__ C, int ldc,
                        const float* __restrict__ row_w, const int* __restrict__ tile_e,
-                       const int* __restrict__ tile_r0, const int* __restrict__ tile_n, int N, int K) {
+                       const int* __restrict__ tile_r0, const int* __restrict__ tile_n, int N, int K,
+                       const CcbGluAct ga, int w_in) {
   ccb::pdl_begin();
   constexpr int KC = 32;
   __shared__ float As[16][KC];
@@ -565,8 +571,10 @@ moe_grouped_f32_kernel(const float* __restrict__ A, int lda, const int* __restri
 #pragma unroll
     for (int r = 0; r < 16; ++r) {
       const float up = __shfl_down_sync(0xffffffffu, acc[r], 1);
-      if (r < n_rows && col + 1 < N && !(col & 1))
-        C[(size_t)(r0 + r) * ldc + (col >> 1)] = acc[r] / (1.f + expf(-acc[r])) * up * row_w[r0 + r];
+      if (r < n_rows && col + 1 < N && !(col & 1)) {
+        const float wr = row_w[r0 + r], wi = w_in ? wr : 1.f, wo = w_in ? 1.f : wr;
+        C[(size_t)(r0 + r) * ldc + (col >> 1)] = glu_act_exact(ga, acc[r] * wi, up * wi) * wo;
+      }
     }
     return;
   }
@@ -663,25 +671,28 @@ CCB_API int ccb_moe_route_sort(const float* logits, int ldl, const float* correc
 
 // mode 0: C (the compute type) [sorted rows, N] = relu(A[src_row] W_e^T)^2 * row_w;  mode 1: C (float) = A W_e^T
 // with A's rows the sorted rows themselves;  mode 2: W_e's N rows are gate and up rows in turn, C (the compute
-// type) [sorted rows, N / 2] = silu(gate) * up * row_w.  Tiles of 16 rows (what moe_sort was given).
+// type) [sorted rows, N / 2] = glu(gate, up) * row_w, or with w_in glu(gate * row_w, up * row_w); limit, alpha, shift,
+// gelu: which glu (CcbGluAct).  Tiles of 16 rows (what moe_sort was given).
 CCB_API int ccb_moe_grouped(const void* A, int lda, const int* src_row, const void* W, int ldw,
                             long long w_expert_stride, void* C, int ldc, const float* row_w, const int* tile_e,
                             const int* tile_r0, const int* tile_n, int max_tiles, int N, int K, int BM, int mode,
-                            int dtype, cudaStream_t stream) {
+                            float limit, float alpha, float shift, int gelu, int w_in, int dtype,
+                            cudaStream_t stream) {
   if (max_tiles <= 0 || N <= 0) return 0;
   if (K <= 0 || mode < 0 || mode > 2 || (mode == 2 && (N & 1))) return CCB_REFUSE_SIZE;
+  const CcbGluAct ga{limit, alpha, shift, gelu};
   if (dtype == CCB_F32) {
     if (BM != 16) return CCB_REFUSE_SIZE;
     dim3 grid(max_tiles, (N + 127) / 128);
     if (mode == 2)
       ccb_launch(moe_grouped_f32_kernel<2>, grid, dim3(128), 0, stream, (const float*)A, lda, src_row, (const float*)W,
-                 ldw, w_expert_stride, (float*)C, ldc, row_w, tile_e, tile_r0, tile_n, N, K);
+                 ldw, w_expert_stride, (float*)C, ldc, row_w, tile_e, tile_r0, tile_n, N, K, ga, w_in);
     else if (mode == 0)
       ccb_launch(moe_grouped_f32_kernel<0>, grid, dim3(128), 0, stream, (const float*)A, lda, src_row, (const float*)W,
-                 ldw, w_expert_stride, (float*)C, ldc, row_w, tile_e, tile_r0, tile_n, N, K);
+                 ldw, w_expert_stride, (float*)C, ldc, row_w, tile_e, tile_r0, tile_n, N, K, ga, w_in);
     else
       ccb_launch(moe_grouped_f32_kernel<1>, grid, dim3(128), 0, stream, (const float*)A, lda, src_row, (const float*)W,
-                 ldw, w_expert_stride, (float*)C, ldc, row_w, tile_e, tile_r0, tile_n, N, K);
+                 ldw, w_expert_stride, (float*)C, ldc, row_w, tile_e, tile_r0, tile_n, N, K, ga, w_in);
     return ccb_launch_status();
   }
   if (dtype != CCB_BF16) return CCB_REFUSE_DTYPE;
@@ -695,13 +706,13 @@ CCB_API int ccb_moe_grouped(const void* A, int lda, const int* src_row, const vo
   dim3 grid16((N + 7) / 8, max_tiles);   // the tiles that hold rows come first in the list, and so do their blocks
   if (mode == 2)
     ccb_launch(moe_grouped_rows16_kernel<2>, grid16, dim3(128), 0, stream, (const __nv_bfloat16*)A, lda, src_row,
-               (const __nv_bfloat16*)W, ldw, w_expert_stride, C, ldc, row_w, tile_e, tile_r0, tile_n, N, K);
+               (const __nv_bfloat16*)W, ldw, w_expert_stride, C, ldc, row_w, tile_e, tile_r0, tile_n, N, K, ga, w_in);
   else if (mode == 0)
     ccb_launch(moe_grouped_rows16_kernel<0>, grid16, dim3(128), 0, stream, (const __nv_bfloat16*)A, lda, src_row,
-               (const __nv_bfloat16*)W, ldw, w_expert_stride, C, ldc, row_w, tile_e, tile_r0, tile_n, N, K);
+               (const __nv_bfloat16*)W, ldw, w_expert_stride, C, ldc, row_w, tile_e, tile_r0, tile_n, N, K, ga, w_in);
   else
     ccb_launch(moe_grouped_rows16_kernel<1>, grid16, dim3(128), 0, stream, (const __nv_bfloat16*)A, lda, src_row,
-               (const __nv_bfloat16*)W, ldw, w_expert_stride, C, ldc, row_w, tile_e, tile_r0, tile_n, N, K);
+               (const __nv_bfloat16*)W, ldw, w_expert_stride, C, ldc, row_w, tile_e, tile_r0, tile_n, N, K, ga, w_in);
   return ccb_launch_status();
 }
 
@@ -738,8 +749,10 @@ CCB_API int ccb_moe_combine(void* out, const float* rows, const int* pair_pos, c
 // act [rows, E F + shared] from gu [rows, 2 (E F + shared)] (gate columns, then up columns): see the kernel.
 CCB_API int ccb_moe_dense_glu_act(void* act, int lda, const void* gu, int ldg, const float* dense_w,
                                   const float* shared_gate, int sg_stride, int rows, int E, int F, int shared,
-                                  int dtype, cudaStream_t stream) {
+                                  float limit, float alpha, float shift, int gelu, int w_in, int dtype,
+                                  cudaStream_t stream) {
   if (rows <= 0) return 0;
+  const CcbGluAct ga{limit, alpha, shift, gelu};
   if (E < 0 || F <= 0 || shared < 0 || lda < E * F + shared || ldg < 2 * (E * F + shared)) return CCB_REFUSE_SIZE;
   if (E > 0 && dense_w == nullptr) return CCB_REFUSE_ARG;
   const int width = E * F + shared;
@@ -747,17 +760,17 @@ CCB_API int ccb_moe_dense_glu_act(void* act, int lda, const void* gu, int ldg, c
       ((reinterpret_cast<uintptr_t>(act) | reinterpret_cast<uintptr_t>(gu)) & 15) == 0) {
     const dim3 vgrid((width / 8 + 255) / 256, rows < 65535 ? rows : 65535);
     ccb_launch(moe_dense_glu_act_vec_kernel, vgrid, dim3(256), 0, stream, (__nv_bfloat16*)act, lda,
-               (const __nv_bfloat16*)gu, ldg, dense_w, shared_gate, sg_stride, rows, E, F, shared);
+               (const __nv_bfloat16*)gu, ldg, dense_w, shared_gate, sg_stride, rows, E, F, shared, ga, w_in);
     return ccb_launch_status();
   }
   const size_t total = (size_t)rows * (E * F + shared);
   const int blocks = (int)((total + 255) / 256 < 65535 * 8 ? (total + 255) / 256 : 65535 * 8);
   if (dtype == CCB_F32)
     ccb_launch(moe_dense_glu_act_kernel<float>, dim3(blocks), dim3(256), 0, stream, (float*)act, lda, (const float*)gu,
-               ldg, dense_w, shared_gate, sg_stride, rows, E, F, shared);
+               ldg, dense_w, shared_gate, sg_stride, rows, E, F, shared, ga, w_in);
   else if (dtype == CCB_BF16)
     ccb_launch(moe_dense_glu_act_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (__nv_bfloat16*)act, lda,
-               (const __nv_bfloat16*)gu, ldg, dense_w, shared_gate, sg_stride, rows, E, F, shared);
+               (const __nv_bfloat16*)gu, ldg, dense_w, shared_gate, sg_stride, rows, E, F, shared, ga, w_in);
   else
     return CCB_REFUSE_DTYPE;
   return ccb_launch_status();

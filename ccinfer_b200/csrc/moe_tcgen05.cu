@@ -9,7 +9,8 @@
 //   * the weight operand is ONE tensor map over all experts' matrices, and the expert moves the box: down the
 //     rows (the first matrices, stacked [E F, D]) or along the columns (the second ones, side by side [D, E F];
 //     what a box reads beyond the expert's F columns meets zeros of A, whose map ends at F);
-//   * the epilogue of the first product is relu(c)^2 * weight(row) in bfloat16, that of the second float.
+//   * the epilogue of the first product is relu(c)^2 * weight(row) (or a gated activation) in bfloat16, that of the
+//     second float.
 // The rows of A must lie in sorted order, so the tokens are gathered first (moe_gather_rows).
 // Every wait on an mbarrier is bounded as in gemm_tcgen05.cu.
 #include "common.cuh"
@@ -34,13 +35,13 @@ __host__ __device__ constexpr uint32_t instr_desc(int n) {
 
 // MODE 0: B rows at e * F + tile column, C bfloat16 = relu(c)^2 * row_w;  MODE 1: B columns at e * F + k, C float;
 // MODE 2: as MODE 0 with B's rows gate and up rows in turn (F rows an expert, N = F), C bfloat16 [*, N / 2] =
-// silu(gate) * up * row_w.
+// glu(gate, up) * row_w (ccb::glu_act), or with w_in glu(gate * row_w, up * row_w).
 template <int BN, int STAGES, int MODE>
 __global__ void __launch_bounds__(kThreadsTc, 1)
 moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                       void* __restrict__ Cout, int ldc, const float* __restrict__ row_w,
                       const int* __restrict__ tile_e, const int* __restrict__ tile_r0,
-                      const int* __restrict__ tile_n, int N, int K, int F, int* status) {
+                      const int* __restrict__ tile_n, int N, int K, int F, const CcbGluAct ga, int w_in, int* status) {
   ccb::pdl_begin();
   const int n_rows = tile_n[blockIdx.x];
   if (n_rows <= 0) return;   // (the whole block, before anything is set up)
@@ -121,6 +122,7 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
       const size_t g = (size_t)(r0 + row);
       const bool mine = row < n_rows;
       const float wr = (MODE != 1 && mine) ? row_w[g] : 1.f;
+      const float wi = w_in ? wr : 1.f, wo = w_in ? 1.f : wr;
 #pragma unroll 1
       for (int c0 = 0; c0 < BN; c0 += 16) {
         uint32_t v[16];
@@ -152,8 +154,8 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
           for (int i = 0; i < 4; ++i) {
             const float g0 = __uint_as_float(v[4 * i]), u0 = __uint_as_float(v[4 * i + 1]);
             const float g1 = __uint_as_float(v[4 * i + 2]), u1 = __uint_as_float(v[4 * i + 3]);
-            const __nv_bfloat162 h = __floats2bfloat162_rn(g0 / (1.f + __expf(-g0)) * u0 * wr,
-                                                           g1 / (1.f + __expf(-g1)) * u1 * wr);
+            const __nv_bfloat162 h = __floats2bfloat162_rn(glu_act(ga, g0 * wi, u0 * wi) * wo,
+                                                           glu_act(ga, g1 * wi, u1 * wi) * wo);
             p[i] = *reinterpret_cast<const uint32_t*>(&h);
           }
           if (n_valid == 16 && (reinterpret_cast<uintptr_t>(dst) & 15) == 0) {
@@ -198,8 +200,8 @@ moe_gather_rows_kernel(uint4* __restrict__ out, const uint4* __restrict__ x, con
 
 template <int MODE>
 int launch(const CUtensorMap& tmA, const CUtensorMap& tmB, void* C, int ldc, const float* row_w, const int* tile_e,
-           const int* tile_r0, const int* tile_n, int max_tiles, int N, int K, int F, int* status,
-           cudaStream_t stream) {
+           const int* tile_r0, const int* tile_n, int max_tiles, int N, int K, int F, const CcbGluAct& ga, int w_in,
+           int* status, cudaStream_t stream) {
   constexpr int BN = 256, STAGES = 4;
   constexpr size_t smem = (size_t)STAGES * (A_STAGE_BYTES + BN * BK * 2) + (2 * STAGES + 1) * 8 + 16 + 1024;
   static bool configured = false;
@@ -210,7 +212,7 @@ int launch(const CUtensorMap& tmA, const CUtensorMap& tmB, void* C, int ldc, con
     configured = true;
   }
   ccb_launch(moe_grouped_tc_kernel<BN, STAGES, MODE>, dim3(max_tiles, (N + BN - 1) / BN), dim3(kThreadsTc), smem,
-             stream, tmA, tmB, C, ldc, row_w, tile_e, tile_r0, tile_n, N, K, F, status);
+             stream, tmA, tmB, C, ldc, row_w, tile_e, tile_r0, tile_n, N, K, F, ga, w_in, status);
   return ccb_launch_status();
 }
 
@@ -234,21 +236,23 @@ CCB_API int ccb_moe_gather_rows(void* out, const void* x, const int* src_row, in
 // mode 0: W = the first matrices stacked [w_rows, K] (expert e at row e * F), C bfloat16 [rows, N = F] with
 // relu(.)^2 * row_w;  mode 1: W = the second matrices side by side [N, w_cols] (expert e at column e * F, K = F),
 // C float [rows, N];  mode 2: W = the first matrices stacked with every expert's gate and up rows in turn (F rows an
-// expert, N = F), C bfloat16 [rows, N / 2] = silu(gate) * up * row_w.
+// expert, N = F), C bfloat16 [rows, N / 2] = glu(gate, up) * row_w, or with w_in glu(gate * row_w, up * row_w); limit,
+// alpha, shift, gelu: which glu (CcbGluAct).
 CCB_API int ccb_moe_grouped_tc(const void* A, int lda, int rows, const void* W, int ldw, int w_rows, int w_cols,
                                void* C, int ldc, const float* row_w, const int* tile_e, const int* tile_r0,
-                               const int* tile_n, int max_tiles, int N, int K, int F, int mode, int* status,
-                               cudaStream_t stream) {
+                               const int* tile_n, int max_tiles, int N, int K, int F, int mode, float limit, float alpha,
+                               float shift, int gelu, int w_in, int* status, cudaStream_t stream) {
   if (max_tiles <= 0 || N <= 0 || rows <= 0) return 0;
   if (K <= 0 || (K & 7) || (F & 7) || (lda & 7) || (ldw & 7) || mode < 0 || mode > 2 || (mode == 2 && (N & 1)) ||
       (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(W) & 15))
     return CCB_REFUSE_SIZE;
+  const CcbGluAct ga{limit, alpha, shift, gelu};
   CUtensorMap tmA, tmB;
   if (!ccb_tensor_map_2d(A, rows, K, lda, BK, BM, &tmA) || !ccb_tensor_map_2d(W, w_rows, w_cols, ldw, BK, 256, &tmB))
     return CCB_REFUSE_ARG;
   if (mode == 2)
-    return launch<2>(tmA, tmB, C, ldc, row_w, tile_e, tile_r0, tile_n, max_tiles, N, K, F, status, stream);
+    return launch<2>(tmA, tmB, C, ldc, row_w, tile_e, tile_r0, tile_n, max_tiles, N, K, F, ga, w_in, status, stream);
   if (mode == 0)
-    return launch<0>(tmA, tmB, C, ldc, row_w, tile_e, tile_r0, tile_n, max_tiles, N, K, F, status, stream);
-  return launch<1>(tmA, tmB, C, ldc, row_w, tile_e, tile_r0, tile_n, max_tiles, N, K, F, status, stream);
+    return launch<0>(tmA, tmB, C, ldc, row_w, tile_e, tile_r0, tile_n, max_tiles, N, K, F, ga, w_in, status, stream);
+  return launch<1>(tmA, tmB, C, ldc, row_w, tile_e, tile_r0, tile_n, max_tiles, N, K, F, ga, w_in, status, stream);
 }

@@ -107,6 +107,7 @@ class Engine:
         group_keys: List[tuple] = []
         windows: List[Optional[int]] = []
         chunks: List[Optional[int]] = []
+        kept: List[int] = []
         token_bytes: List[int] = []   # per group: bytes one token costs in all its layers
         owners: Dict[int, object] = {}  # run entry -> its CacheNeed
         self._entry_group: Dict[int, int] = {}
@@ -127,6 +128,7 @@ class Engine:
                     group_keys.append(need.group_key)
                     windows.append(need.window)
                     chunks.append(getattr(need, "chunk", None))
+                    kept.append(getattr(need, "keep_first", 0))
                     token_bytes.append(0)
                 g = group_keys.index(need.group_key)
                 self._entry_group[i] = g
@@ -153,9 +155,10 @@ class Engine:
                 if e.cache_of not in self._entry_group:
                     raise InvalidArgument(f"order[{i}] reads the cache of entry {e.cache_of}, which keeps none")
                 self._entry_group[i] = self._entry_group[e.cache_of]
-        # how many of a request's latest tokens a group holds at most (None: all of them)
-        spans = [min(x for x in (w, c) if x is not None) if (w is not None or c is not None) else None
-                 for w, c in zip(windows, chunks)]
+        # how many tokens of a request a group holds at most between steps: its latest ones and, in whole pages, the
+        # first ones where those are kept (None: all of them)
+        spans = [min(x for x in (w, c) if x is not None) + -(-k // P) * P if (w is not None or c is not None) else None
+                 for w, c, k in zip(windows, chunks, kept)]
         pages = self._pages_per_group(opt, group_keys, spans, token_bytes)
         for i, need in owners.items():
             n = pages[self._entry_group[i]]
@@ -168,7 +171,8 @@ class Engine:
         if plan.max_position is not None:
             limit = min(limit, plan.max_position)
         self.max_context = min(opt.max_context, limit) if opt.max_context else limit
-        self.cache = CacheManager([GroupSpec(k, w, P, n, c) for k, w, n, c in zip(group_keys, windows, pages, chunks)],
+        self.cache = CacheManager([GroupSpec(key, w, P, n, c, k)
+                                   for key, w, n, c, k in zip(group_keys, windows, pages, chunks, kept)],
                                   opt.max_requests, opt.max_tokens_per_step, self.max_context)
         self.graph_safe = all(getattr(p, "graph_safe", True) for p in plan.parts())
 
@@ -218,7 +222,7 @@ class Engine:
         src/worker/worker.cpp:272), or its share of ``kv_memory_fraction`` of the free memory.  A window
         group never needs more than what ``max_requests`` requests can hold at once, the window plus the
         step's new tokens each, and gets no more than that.  ``kv_group_tokens`` sets single groups by their
-        key (("all",) or ("window", W)).
+        key (("all",), ("window", W), ...: ``CacheNeed.group_key``).
         """
         P = opt.page_size
         explicit = dict(opt.kv_group_tokens or {})

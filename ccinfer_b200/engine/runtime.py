@@ -7,7 +7,7 @@ import torch
 
 from .. import kernels
 from ..errors import DeviceFault, ExtensionMissing, ScratchMoved, Unsupported
-from ..parts.base import UnscaledRows
+from ..parts.base import NormedPair, UnscaledRows
 
 
 class ScratchPool:
@@ -74,8 +74,8 @@ class Runtime:
 
     @staticmethod
     def rows(x):
-        """x as a plain tensor (rows that a norm left short of their factor are finished)."""
-        return x.finish() if isinstance(x, UnscaledRows) else x
+        """x as a plain tensor (rows that a norm left short of their factor are finished, and a pair's sum is made)."""
+        return x.finish() if isinstance(x, (UnscaledRows, NormedPair)) else x
 
     def _into_stream(self, out, x, w, sink) -> bool:
         """The product as the last one of a part, with few rows: added into the residual stream by its own
@@ -168,12 +168,9 @@ class Runtime:
 
         A few tokens in bfloat16 with the blocked layout: one kernel (the activation is the product's
         epilogue).  Otherwise the product into scratch and the activation kernel.
-        ``activation`` ("clamped_glu", limit, alpha, shift): that activation in place of silu(g) * u, in the
-        same epilogues or as a kernel of its own."""
+        ``activation`` (a ``kernels.GluAct``): that activation in place of silu(g) * u, in the same epilogues or as a
+        kernel of its own."""
         if activation is not None:
-            kind, limit, alpha, shift = activation
-            if kind != "clamped_glu":
-                raise Unsupported(f"gated activation {kind!r}")
             x = self.rows(x)
             M, K = x.shape
             N = w.shape[0]
@@ -188,11 +185,11 @@ class Runtime:
             elif (blocked and M >= kernels.PAIR_SWIGLU_MIN_ROWS and N % 128 == 0 and kernels.gemm_tc_fits(K, x, w)):
                 fused = "pair"
             if fused is not None:
-                kernels.gemm_glu_bf16(act, x, w, limit, alpha, shift, fused, status=self.status)
+                kernels.gemm_glu_bf16(act, x, w, activation, fused, status=self.status)
                 return act
             gu = self.scratch.get("ffn_gate_up", (self.max_tokens, N), self.dtype)[:M]
             self.linear(gu, x, w)
-            kernels.clamped_glu(act, gu, block, limit, alpha, shift)
+            kernels.gated_act(act, gu, block, activation)
             return act
         un = x if isinstance(x, UnscaledRows) else None
         if un is not None:

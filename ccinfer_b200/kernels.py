@@ -39,11 +39,11 @@ _SIGNATURES = {
     "ccb_gemm_tc_swiglu_bf16": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                                 c_void_p],
     "ccb_gemm_tc_glu_bf16": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-                             c_float, c_void_p, c_void_p],
+                             c_float, c_int, c_void_p, c_void_p],
     "ccb_gemm_fewrows_glu_bf16": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                  c_float, c_float, c_float, c_void_p, c_void_p],
+                                  c_float, c_float, c_float, c_int, c_void_p, c_void_p],
     "ccb_gemm_tc_pair_glu_bf16": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                  c_float, c_float, c_int, c_void_p, c_void_p],
+                                  c_float, c_float, c_int, c_int, c_void_p, c_void_p],
     "ccb_gemm_fewrows_set_stages": [c_int],
     "ccb_gemm_fewrows_bf16": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                               c_void_p, c_void_p],
@@ -66,7 +66,7 @@ _SIGNATURES = {
                                    c_void_p, c_float, c_int, c_void_p, c_void_p],
     "ccb_postnorm_residual": [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_void_p, c_float,
                               c_int, c_int, c_int, c_void_p],
-    "ccb_clamped_glu": [c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p],
+    "ccb_gated_act": [c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_int, c_void_p],
     "ccb_delta_prepare": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p,
                           c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p],
@@ -92,7 +92,7 @@ _SIGNATURES = {
     "ccb_moe_route": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                       c_int, c_int, c_int, c_float, c_void_p],
     "ccb_moe_dense_glu_act": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                              c_int, c_void_p],
+                              c_float, c_float, c_float, c_int, c_int, c_int, c_void_p],
     "ccb_conv_rows": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                       c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p,
                       c_void_p],
@@ -100,18 +100,21 @@ _SIGNATURES = {
                             c_void_p],
     "ccb_attention_split_ex": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                               c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
+                               c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
     "ccb_moe_dense_act": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "ccb_moe_sort": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                      c_void_p, c_void_p, c_void_p],
-    "ccb_moe_route_sort": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+    "ccb_moe_route_sort": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                           c_int,
                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float,
                            c_void_p],
     "ccb_moe_grouped": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
-                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int,
+                        c_int, c_int, c_void_p],
     "ccb_moe_gather_rows": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "ccb_moe_grouped_tc": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p,
-                           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+                           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int,
+                           c_int, c_void_p, c_void_p],
     "ccb_moe_combine": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "ccb_scaled_residual": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_void_p],
     "ccb_concat_cast": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
@@ -128,24 +131,25 @@ _SIGNATURES = {
     "ccb_attention_split": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
                             c_int, c_void_p, c_void_p],
-    # (the four arguments before the status word: chunk, sink, gate, gate_stride)
+    # (the five arguments before the status word: chunk, keep, sink, gate, gate_stride)
     "ccb_attention_decode_mma": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                 c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+                                 c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
     "ccb_attention_decode_tma": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                 c_float, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+                                 c_float, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p,
+                                 c_void_p],
     "ccb_attention_decode_tma_fused": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                        c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int,
-                                       c_void_p, c_float, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int,
+                                       c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
                                        c_void_p, c_void_p],
     "ccb_attention_prefill_mma": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                   c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
-                                     c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+                                  c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
     "ccb_attention_prefill_tc": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                  c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
-                                 c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+                                 c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
     "ccb_gemm_f32": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "ccb_cublas_create": [ctypes.POINTER(c_void_p)],
     "ccb_cublas_destroy": [c_void_p],
@@ -174,6 +178,15 @@ _SIGNATURES = {
     "ccb_attention_talking_mma_fits": [c_int, c_int, c_int],
     "ccb_attention_talking_mma": [c_void_p] * 8 + [c_int] * 10 + [c_void_p, c_void_p, c_int, c_void_p, c_void_p],
     "ccb_embed_pair": [c_void_p] * 10 + [c_float] + [c_int] * 9 + [c_void_p, c_int, c_void_p, c_void_p],
+    "ccb_norm_chain": [c_void_p] * 6 + [c_float] * 3 + [c_int, c_void_p, c_void_p, c_float, c_float, c_void_p]
+                      + [c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+    "ccb_qk_rows": [c_void_p, c_int] + [c_void_p] * 4 + [c_int] + [c_void_p] * 3 + [c_float, c_int] + [c_void_p] * 6
+                   + [c_int] * 9 + [c_void_p, c_void_p],
+    "ccb_memory_prepare": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                           c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p],
+    "ccb_memory_gates": [c_void_p, c_int, c_void_p, c_void_p, c_float] + [c_void_p] * 6 + [c_int] * 3 + [c_void_p],
+    "ccb_memory_output": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int,
+                          c_float, c_int, c_void_p],
     "ccb_relu_squared": [c_void_p, c_void_p, c_longlong, c_int, c_void_p],
     "ccb_scaled_sum": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_longlong, c_int, c_void_p],
     "ccb_sample_rows": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
@@ -369,8 +382,30 @@ def gemm_tc_swiglu_bf16(act, a, w, status=None) -> None:
                                          _p(status), _stream()), "gemm_tc_swiglu_bf16")
 
 
-def gemm_glu_bf16(act, a, w, limit: float, alpha: float, shift: float, kind: str, status=None) -> None:
-    """act[M, F] = glu(a Wg^T, a Wu^T) with the clamped activation of ``clamped_glu`` as the epilogue of the
+class GluAct:
+    """A gated activation of the products' epilogues (``ccb::glu_act``): ``GluAct()`` silu(g) * u;
+    ``GluAct.clamped(limit, alpha, shift)`` min(g, limit) * sigmoid(alpha min(g, limit)) * (clamp(u, -limit, limit) +
+    shift); ``GluAct.gelu_tanh()`` gelu(g) * u with the tanh form of gelu."""
+
+    def __init__(self, limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0, gelu: bool = False):
+        self.args = (float(limit), float(alpha), float(shift), 1 if gelu else 0)
+
+    @classmethod
+    def clamped(cls, limit: float, alpha: float, shift: float) -> "GluAct":
+        if not limit > 0:
+            raise Unsupported("the clamped activation's limit must be > 0")
+        return cls(limit, alpha, shift)
+
+    @classmethod
+    def gelu_tanh(cls) -> "GluAct":
+        return cls(gelu=True)
+
+
+_SILU_GLU = GluAct()
+
+
+def gemm_glu_bf16(act, a, w, glu: GluAct, kind: str, status=None) -> None:
+    """act[M, F] = glu(a Wg^T, a Wu^T) with another activation than silu(g) * u as the epilogue of the
     product, w [2F, K] interleaved in blocks of SWIGLU_BLOCK rows.  ``kind``: "tc" (tcgen05, M <= 16),
     "fewrows" (TMA ring, M <= 16) or "pair" (tcgen05 on pairs of SMs, many rows)."""
     _cuda(w, status)
@@ -379,7 +414,7 @@ def gemm_glu_bf16(act, a, w, limit: float, alpha: float, shift: float, kind: str
     F = act.shape[1]
     assert w.shape == (2 * F, K) and act.shape[0] == M and F % SWIGLU_BLOCK == 0
     assert a.stride(1) == 1 and w.stride(1) == 1 and act.stride(1) == 1
-    args = (float(limit), float(alpha), float(shift))
+    args = glu.args
     if kind == "tc":
         rc = lib().ccb_gemm_tc_glu_bf16(_p(act), _p(a), _p(w), M, F, K, a.stride(0), w.stride(0), act.stride(0),
                                         *args, _p(status), _stream())
@@ -494,14 +529,17 @@ def postnorm_residual(h, delta, w_post, mult: float, eps_post: float, add=None, 
                                        _stream()), "postnorm_residual")
 
 
-def clamped_glu(act, gate_up, block: int, limit: float, alpha: float, up_shift: float) -> None:
-    """act = g * sigmoid(alpha g) * (u + up_shift) with g = min(gate, limit), u = clamp(up, -limit, limit);
-    the layouts of gate_up are those of ``silu_mul``."""
+def gated_act(act, gate_up, block: int, glu: GluAct) -> None:
+    """act = glu(gate, up), any activation but silu(g) * u; the layouts of gate_up are those of ``silu_mul``."""
     _cuda(act, gate_up)
     T, F = act.shape
     assert gate_up.shape == (T, 2 * F) and act.dtype == gate_up.dtype
-    _check(lib().ccb_clamped_glu(_p(act), _p(gate_up), T, F, int(block), float(limit), float(alpha),
-                                 float(up_shift), _dt(act), _stream()), "clamped_glu")
+    _check(lib().ccb_gated_act(_p(act), _p(gate_up), T, F, int(block), *glu.args, _dt(act), _stream()), "gated_act")
+
+
+def clamped_glu(act, gate_up, block: int, limit: float, alpha: float, up_shift: float) -> None:
+    """``gated_act`` with g * sigmoid(alpha g) * (u + up_shift), g = min(gate, limit), u = clamp(up, -limit, limit)."""
+    gated_act(act, gate_up, block, GluAct.clamped(limit, alpha, up_shift))
 
 
 def delta_prepare(proj, offsets, a, conv_w, taps: int, conv_state, A_log, dt_bias, entry_of_token, cu_q, state_slot,
@@ -733,8 +771,10 @@ def moe_route(logits, correction, idx, wts, dense_w, groups: int, keep: int, rul
                                int(groups), int(keep), top, *(rule or _PLAIN_ROUTE).args, _stream()), "moe_route")
 
 
-def moe_dense_glu_act(act, gu, dense_w, E: int, F: int, shared: int, shared_gate=None) -> None:
-    """act [T, E F + shared] = silu(gate) * up * weight from the rows ``gu`` [T, 2 (E F + shared)] of ONE product
+def moe_dense_glu_act(act, gu, dense_w, E: int, F: int, shared: int, shared_gate=None, glu: GluAct = None,
+                      weight_in: bool = False) -> None:
+    """act [T, E F + shared] = glu(gate, up) * weight (``glu`` None: silu(gate) * up), or with ``weight_in``
+    glu(gate * weight, up * weight), from the rows ``gu`` [T, 2 (E F + shared)] of ONE product
     over all experts' gate rows and then all their up rows: weight = dense_w[t, e] for expert e's columns (exact
     zeros where it was not chosen); the ``shared`` columns after them get sigmoid(shared_gate[t]) (``shared_gate``
     a float column view [T], or None for 1)."""
@@ -747,7 +787,7 @@ def moe_dense_glu_act(act, gu, dense_w, E: int, F: int, shared: int, shared_gate
                                    and shared_gate.dim() == 1)
     _check(lib().ccb_moe_dense_glu_act(_p(act), act.stride(0), _p(gu), gu.stride(0), _p(dense_w), _p(shared_gate),
                                        shared_gate.stride(0) if shared_gate is not None else 0, T, E, F, shared,
-                                       _dt(act), _stream()), "moe_dense_glu_act")
+                                       *(glu or _SILU_GLU).args, 1 if weight_in else 0, _dt(act), _stream()), "moe_dense_glu_act")
 
 
 def moe_dense_act(act, dense_w, E: int, F: int, shared: int) -> None:
@@ -801,18 +841,19 @@ def moe_route_sort(logits, correction, idx, wts, groups: int, keep: int, E: int,
 
 
 def moe_grouped(c, a, src_row, w, w_expert_stride: int, row_w, tile_e, tile_r0, tile_n, N: int, K: int, BM: int,
-                mode: int) -> None:
+                mode: int, glu: GluAct = None, weight_in: bool = False) -> None:
     """The product of every tile's rows with its expert's matrix (``w`` [*, ldw] viewed from the first expert's
     first element, expert e at + e * w_expert_stride elements, N rows of K).  mode 0: c[row] = relu(a[src_row[row]]
     W_e^T)^2 * row_w[row] in the compute type; mode 1: c[row] = a[row] W_e^T in float; mode 2: W_e's rows are gate
-    and up rows in turn (N of them), c[row] [N / 2] = silu(gate) * up * row_w[row] in the compute type."""
+    and up rows in turn (N of them), c[row] [N / 2] = glu(gate, up) * row_w[row] (``glu`` None: silu(gate) * up) in the
+    compute type, or with ``weight_in`` glu(gate * row_w[row], up * row_w[row])."""
     _cuda(src_row, row_w, tile_e, tile_r0, tile_n)
     assert a.stride(1) == 1 and w.stride(1) == 1 and c.stride(1) == 1 and a.dtype == w.dtype
     assert c.dtype == (torch.float32 if mode == 1 else a.dtype) and a.shape[1] == K
     assert c.shape[1] == (N // 2 if mode == 2 else N)
     _check(lib().ccb_moe_grouped(_p(a), a.stride(0), _p(src_row), _p(w), w.stride(0), int(w_expert_stride), _p(c),
                                  c.stride(0), _p(row_w), _p(tile_e), _p(tile_r0), _p(tile_n), tile_e.numel(), N, K, BM,
-                                 mode, _dt(a), _stream()), "moe_grouped")
+                                 mode, *(glu or _SILU_GLU).args, 1 if weight_in else 0, _dt(a), _stream()), "moe_grouped")
 
 
 MOE_TC_ROWS = 128   # rows of a tile of the tcgen05 grouped product
@@ -828,18 +869,19 @@ def moe_gather_rows(out, x, src_row) -> None:
            "moe_gather_rows")
 
 
-def moe_grouped_tc(c, a, w, row_w, tile_e, tile_r0, tile_n, N: int, K: int, F: int, mode: int, status=None) -> None:
+def moe_grouped_tc(c, a, w, row_w, tile_e, tile_r0, tile_n, N: int, K: int, F: int, mode: int, status=None,
+                   glu: GluAct = None, weight_in: bool = False) -> None:
     """``moe_grouped`` on tcgen05 tensor cores for tiles of MOE_TC_ROWS sorted rows (bfloat16).  ``a`` holds the
     sorted rows themselves.  mode 0: ``w`` = all first matrices stacked [E F, K], c bfloat16 [rows, F] =
     relu(a W_e^T)^2 * row_w;  mode 1: ``w`` = all second matrices side by side [N, E F] (K = F), c float;  mode 2:
-    as mode 0 with every expert's F = N rows gate and up rows in turn, c bfloat16 [rows, N / 2] = silu(gate) * up *
-    row_w."""
+    as mode 0 with every expert's F = N rows gate and up rows in turn, c bfloat16 [rows, N / 2] as ``moe_grouped``'s."""
     _cuda(a, w, row_w, tile_e, tile_r0, tile_n, status)
     assert a.dtype == w.dtype == torch.bfloat16 and c.dtype == (torch.float32 if mode == 1 else torch.bfloat16)
     assert a.shape[1] == K and c.shape == (a.shape[0], N // 2 if mode == 2 else N) and c.is_contiguous()
     _check(lib().ccb_moe_grouped_tc(_p(a), a.stride(0), a.shape[0], _p(w), w.stride(0), w.shape[0], w.shape[1], _p(c),
                                     c.stride(0), _p(row_w), _p(tile_e), _p(tile_r0), _p(tile_n), tile_e.numel(), N, K,
-                                    F, mode, _p(status), _stream()), "moe_grouped_tc")
+                                    F, mode, *(glu or _SILU_GLU).args, 1 if weight_in else 0, _p(status), _stream()),
+           "moe_grouped_tc")
 
 
 def moe_combine(out, rows, pair_pos, shared, top: int) -> None:
@@ -885,6 +927,133 @@ def embed_pair(h, rows, table, pair_table, ids, positions, entry_of_token, cu_q,
                                 _p(status), _stream()), "embed_pair")
     if pair_table is not None:
         counters.own += 1   # the kernel that stores each request's last token
+
+
+class NormSpec:
+    """A norm as ``norm_chain`` takes it: ``kind`` "rms" (weight) or "layer" (weight and bias)."""
+
+    def __init__(self, kind: str, weight, bias, eps: float):
+        assert kind in ("rms", "layer") and (kind == "rms") == (bias is None)
+        self.kind, self.weight, self.bias, self.eps = kind, weight, bias, float(eps)
+
+    @property
+    def args(self):
+        return (1 if self.kind == "rms" else 2, _p(self.weight), _p(self.bias), self.eps)
+
+
+def _norm_args(spec, D: int):
+    if spec is None:
+        return (0, None, None, 0.0)
+    _cuda(spec.weight, spec.bias)
+    assert spec.weight.dtype == torch.float32 and spec.weight.numel() == D
+    assert spec.bias is None or (spec.bias.dtype == torch.float32 and spec.bias.numel() == D)
+    return spec.args
+
+
+def norm_chain(h, delta=None, post: NormSpec = None, nxt: NormSpec = None, y=None, mult: float = 1.0, add=None, pair=None,
+               row_idx=None, n_rows: int = None, status=None) -> None:
+    """h += mult * post(d) [+ add];  y = nxt(h), or the stream's own rows with ``nxt`` None, in one pass over each row.
+
+    d is ``delta``, or with ``pair`` = (delta_b, wa, wb, ca, cb, eps) the sum ca * unit(delta) * wa + cb *
+    unit(delta_b) * wb of two outputs over their root mean squares.  h and add float [T, D]; delta, delta_b and y of
+    the storage type; norm weights float [D].  ``row_idx`` (int32): only those rows, h is left as it is."""
+    _cuda(h, delta, add, y, row_idx, status)
+    T, D = h.shape
+    assert h.dtype == torch.float32 and (delta is None or delta.shape == (T, D))
+    assert add is None or (add.dtype == torch.float32 and add.shape[1] == D and add.shape[0] >= T)
+    rows = T if row_idx is None else (row_idx.numel() if n_rows is None else int(n_rows))
+    assert y is None or (y.shape[0] >= rows and y.shape[1] == D and (delta is None or delta.dtype == y.dtype))
+    assert nxt is None or y is not None
+    second = wa = wb = None
+    ca = cb = eps = 0.0
+    if pair is not None:
+        second, wa, wb, ca, cb, eps = pair
+        _cuda(second, wa, wb)
+        assert delta is not None and second.shape == (T, D) and second.dtype == delta.dtype
+        assert wa.dtype == wb.dtype == torch.float32 and wa.numel() == wb.numel() == D
+    ref = delta if delta is not None else y
+    _check(lib().ccb_norm_chain(_p(y), _p(h), _p(delta), _p(second), _p(wa), _p(wb), float(ca), float(cb), float(eps),
+                                *_norm_args(post, D), float(mult), _p(add), *_norm_args(nxt, D), _p(row_idx), rows, T, D,
+                                _dt(ref) if ref is not None else F32, _p(status), _stream()), "norm_chain")
+
+
+def qk_rows(rows, q_out, k_cache, v_cache, conv_w, taps: int, state, q_w, k_w, eps: float, n_real: int, inv_freq,
+            positions, slot_map, entry_of_token, cu_q, state_slot, n_entries: int, status=None) -> None:
+    """From the rows of a q | k product [T, (nq + nkv) * hd] to the queries ``q_out`` [T, nq, hd] and the cached keys
+    and values, where the values are the keys as the convolution leaves them and the norms of q and k run over the
+    whole projection (``qk_rows.cu``).  ``conv_w`` float [taps, channels] or None; ``state`` [slots, taps - 1,
+    channels]; ``q_w`` [nq * hd] and ``k_w`` [nkv * hd] float or None; ``n_real`` the channels of a head that count in
+    the norms' means.  Requests that bring several tokens have their state moved on by ``conv_state_rows``."""
+    _cuda(q_out, k_cache, v_cache, conv_w, state, q_w, k_w, inv_freq, positions, slot_map, entry_of_token, cu_q, state_slot,
+          status)
+    T, nq, hd = q_out.shape
+    num_pages, nkv, page_size, hd2 = k_cache.shape
+    C = (nq + nkv) * hd
+    assert rows.is_cuda and rows.stride(1) == 1 and rows.shape[0] == T and rows.shape[1] >= C and hd2 == hd
+    assert rows.dtype == q_out.dtype == k_cache.dtype == v_cache.dtype and v_cache.shape == k_cache.shape
+    assert conv_w is None or (conv_w.dtype == torch.float32 and conv_w.shape == (taps, C))
+    assert taps == 1 or (state is not None and state.dtype == rows.dtype and tuple(state.shape[1:]) == (taps - 1, C))
+    assert all(w is None or (w.dtype == torch.float32 and w.numel() == n) for w, n in
+               ((q_w, nq * hd), (k_w, nkv * hd), (inv_freq, hd // 2)))
+    _check(lib().ccb_qk_rows(_p(rows), rows.stride(0), _p(q_out), _p(k_cache), _p(v_cache), _p(conv_w), int(taps), _p(state),
+                             _p(q_w), _p(k_w), float(eps), int(n_real), _p(inv_freq), _p(positions), _p(slot_map),
+                             _p(entry_of_token), _p(cu_q), _p(state_slot), T, int(n_entries),
+                             state.shape[0] if state is not None else 0, nq, nkv, hd, page_size, num_pages * page_size,
+                             _dt(rows), _p(status), _stream()), "qk_rows")
+
+
+def memory_prepare(proj, offsets, inv_freq, rot_dims: int, positions, qn, kn, vv, H: int, dk: int, dv: int, q_mult: float,
+                   k_mult: float, ones: bool = False) -> None:
+    """Float rows of a matrix memory's q and k [T, H, dk] (rotated in pairs (i, i + rot_dims / 2) where ``rot_dims`` >
+    0, then times ``q_mult`` / ``k_mult``) and v [T, H, dv (+ 1 with ``ones``: a last column of ones)] from the
+    projection's columns at ``offsets`` (q, k, v)."""
+    _cuda(inv_freq, positions, qn, kn, vv)
+    T = qn.shape[0]
+    assert proj.is_cuda and proj.stride(1) == 1 and proj.shape[0] == T
+    assert qn.dtype == kn.dtype == vv.dtype == torch.float32 and qn.shape == kn.shape == (T, H, dk)
+    assert vv.shape == (T, H, dv + (1 if ones else 0)) and (rot_dims == 0 or inv_freq.numel() >= rot_dims // 2)
+    oq, ok, ov = offsets
+    assert max(oq + H * dk, ok + H * dk, ov + H * dv) <= proj.shape[1]
+    _check(lib().ccb_memory_prepare(_p(proj), proj.stride(0), oq, ok, ov, _p(inv_freq), int(rot_dims), _p(positions), _p(qn),
+                                    _p(kn), _p(vv), T, H, dk, dv, float(q_mult), float(k_mult), 1 if ones else 0, _dt(proj),
+                                    _stream()), "memory_prepare")
+
+
+def memory_gates(z, bias_i, bias_f, cap: float, m_state, cu_q, state_slot, decay, put, floor, n_entries: int,
+                 H: int) -> None:
+    """The exponential gates of a matrix memory with their running maximum (``scalar_memory.cu``): ``z`` float [T, 2 H]
+    pre-activations (input gates, forget gates); ``m_state`` float [slots, H] is moved on; decay, put and floor float
+    [T, H] are exp(f + m_before - m), exp(i - m) and exp(-m)."""
+    _cuda(bias_i, bias_f, m_state, cu_q, state_slot, decay, put, floor)
+    assert z.dtype == torch.float32 and z.stride(1) == 1 and z.shape[1] >= 2 * H and m_state.dtype == torch.float32
+    assert decay.shape == put.shape == floor.shape == (z.shape[0], H) and decay.dtype == torch.float32
+    _check(lib().ccb_memory_gates(_p(z), z.stride(0), _p(bias_i), _p(bias_f), float(cap), _p(m_state), _p(cu_q),
+                                  _p(state_slot), _p(decay), _p(put), _p(floor), int(n_entries), H, m_state.shape[0],
+                                  _stream()), "memory_gates")
+
+
+def memory_recurrence(qn, kn, vv, decay, put, state, out, cu_q, state_slot, n_entries: int, H: int, dk: int,
+                      dv: int) -> None:
+    """S <- a_t S + b_t k_t v_t^T, o_t = S^T q_t with one decay a_t (``decay`` float [T, H]) and one factor on the
+    write (``put`` float [T, H], None: 1) per head and token; S is ``state`` float [slots, H, dv, dk]."""
+    _cuda(qn, kn, vv, decay, put, state, out, cu_q, state_slot)
+    _check(lib().ccb_ssm_recurrence(_p(qn), _p(kn), _p(vv), _p(decay), _p(put), _p(state), _p(out), _p(cu_q),
+                                    _p(state_slot), int(n_entries), H, H, dk, dv, _stream()), "memory_recurrence")
+
+
+def memory_output(y, o, gate, H: int, dv: int, eps: float, weight=None, floor=None, den_eps: float = 0.0,
+                  silu_gate: bool = False) -> None:
+    """y [T, H dv] = unit(o / den) * weight * act(gate) per head: ``o`` float [T, H, dv], or with ``floor`` (float
+    [T, H], exp(-m)) [T, H, dv + 1] whose last column n . q gives den = max(|n . q|, floor) + den_eps; ``weight`` float
+    [H dv] or None; act is sigmoid, or silu with ``silu_gate``; ``gate`` the gate's columns (compute type)."""
+    _cuda(y, o, weight, floor)
+    T = y.shape[0]
+    assert y.shape == (T, H * dv) and o.shape == (T, H, dv + (1 if floor is not None else 0)) and o.dtype == torch.float32
+    assert gate.dtype == y.dtype and gate.stride(1) == 1 and gate.shape[0] == T and gate.shape[1] >= H * dv
+    assert weight is None or (weight.dtype == torch.float32 and weight.numel() == H * dv)
+    _check(lib().ccb_memory_output(_p(y), _p(o), _p(floor), float(den_eps), _p(gate), gate.stride(0),
+                                   1 if silu_gate else 0, _p(weight), T, H, dv, float(eps), _dt(y), _stream()),
+           "memory_output")
 
 
 def relu_squared(act, x) -> None:
@@ -1117,11 +1286,12 @@ def attention_split_plan(n_rows: int, nq: int, nkv: int, hd: int, heads_per_bloc
 
 def attention_split(q, k_cache, v_cache, out, part_acc, part_ml, positions, entry_of_token, block_table,
                     n_entries: int, row0: int, n_rows: int, window: int, scale: float, num_splits: int,
-                    status=None, chunk: int = 0, sink=None, gate=None) -> None:
+                    status=None, chunk: int = 0, sink=None, gate=None, keep: int = 0) -> None:
     """Attention of the token rows row0 .. row0 + n_rows - 1, each a single query with its own position
     and request; the key range is cut into ``num_splits`` pieces merged afterwards (scratch from
     ``attention_split_plan``; unused with one split).  ``chunk`` > 0: a query sees only the keys of its own run of
-    ``chunk`` positions (counted from the sequence's start); ``sink`` float [nq]: one more term exp(sink[h]) in
+    ``chunk`` positions (counted from the sequence's start); ``keep`` > 0: the first ``keep`` keys of the sequence
+    are seen whatever the window and the chunk leave out; ``sink`` float [nq]: one more term exp(sink[h]) in
     every softmax denominator of head h; ``gate`` [T, >= nq] (compute type, a view with unit column stride): head
     h's result times sigmoid(gate[t, h])."""
     _cuda(q, k_cache, v_cache, out, part_acc, part_ml, positions, entry_of_token, block_table, status, sink)
@@ -1138,7 +1308,7 @@ def attention_split(q, k_cache, v_cache, out, part_acc, part_ml, positions, entr
     _check(lib().ccb_attention_split_ex(_p(q), _p(k_cache), _p(v_cache), _p(out), _p(part_acc), _p(part_ml),
                                         _p(positions), _p(entry_of_token), _p(block_table), block_table.stride(0),
                                         n_entries, row0, n_rows, nq, nkv, hd, page_size, num_pages, int(window),
-                                        float(scale), num_splits, int(chunk), _p(sink), _p(gate),
+                                        float(scale), num_splits, int(chunk), int(keep), _p(sink), _p(gate),
                                         gate.stride(0) if gate is not None else 0, _dt(q), _p(status), _stream()),
            "attention_split")
     if num_splits > 1:
@@ -1149,18 +1319,19 @@ DECODE_MMA_HEAD_SIZES = (64, 128)
 DECODE_MMA_HEADS_PER_BLOCK = 16
 
 
-def _attn_extra(q_rows: int, nq: int, dtype, chunk: int, sink, gate):
-    """The four arguments ``chunk, sink, gate, gate_stride`` of the attention kernels (see ``attention_split``)."""
+def _attn_extra(q_rows: int, nq: int, dtype, chunk: int, sink, gate, keep: int = 0):
+    """The five arguments ``chunk, keep, sink, gate, gate_stride`` of the attention kernels (see
+    ``attention_split``)."""
     _cuda(sink)   # (the gate's rows are a view into a wider row)
-    assert chunk >= 0 and (sink is None or (sink.dtype == torch.float32 and sink.numel() == nq))
+    assert chunk >= 0 and keep >= 0 and (sink is None or (sink.dtype == torch.float32 and sink.numel() == nq))
     assert gate is None or (gate.is_cuda and gate.dtype == dtype and gate.stride(1) == 1 and gate.shape[0] == q_rows
                             and gate.shape[1] >= nq)
-    return int(chunk), _p(sink), _p(gate), gate.stride(0) if gate is not None else 0
+    return int(chunk), int(keep), _p(sink), _p(gate), gate.stride(0) if gate is not None else 0
 
 
 def attention_decode_mma(q, k_cache, v_cache, out, part_acc, part_ml, positions, entry_of_token, block_table,
                          n_entries: int, row0: int, n_rows: int, window: int, scale: float, num_splits: int,
-                         status=None, chunk: int = 0, sink=None, gate=None) -> None:
+                         status=None, chunk: int = 0, sink=None, gate=None, keep: int = 0) -> None:
     """As attention_split, on tensor cores: bfloat16, head size 64 or 128, a block per (row, kv head, split)
     serving the whole group of q heads."""
     _cuda(q, k_cache, v_cache, out, part_acc, part_ml, positions, entry_of_token, block_table, status)
@@ -1176,7 +1347,7 @@ def attention_decode_mma(q, k_cache, v_cache, out, part_acc, part_ml, positions,
                                           _p(positions), _p(entry_of_token), _p(block_table),
                                           block_table.stride(0), n_entries, row0, n_rows, nq, nkv, hd, page_size,
                                           num_pages, int(window), float(scale), num_splits,
-                                          *_attn_extra(T, nq, q.dtype, chunk, sink, gate), _p(status),
+                                          *_attn_extra(T, nq, q.dtype, chunk, sink, gate, keep), _p(status),
                                           _stream()), "attention_decode_mma")
     if num_splits > 1:
         counters.own += 1  # the merge kernel
@@ -1188,7 +1359,7 @@ def attention_decode_tma_fits(hd: int, page_size: int) -> bool:
 
 def attention_decode_tma(q, k_cache, v_cache, out, part_acc, part_ml, positions, entry_of_token, block_table,
                          n_entries: int, row0: int, n_rows: int, window: int, scale: float, num_splits: int,
-                         status=None, merge_counters=None, chunk: int = 0, sink=None, gate=None) -> None:
+                         status=None, merge_counters=None, chunk: int = 0, sink=None, gate=None, keep: int = 0) -> None:
     """As attention_decode_mma, with keys and values loaded page by page through TMA boxes by a producer warp
     (page size a power of two from 8 to 64).
 
@@ -1213,7 +1384,7 @@ def attention_decode_tma(q, k_cache, v_cache, out, part_acc, part_ml, positions,
                                           _p(positions), _p(entry_of_token), _p(block_table),
                                           block_table.stride(0), n_entries, row0, n_rows, nq, nkv, hd, page_size,
                                           num_pages, int(window), float(scale), num_splits, _p(merge_counters),
-                                          *_attn_extra(T, nq, q.dtype, chunk, sink, gate), _p(status), _stream()),
+                                          *_attn_extra(T, nq, q.dtype, chunk, sink, gate, keep), _p(status), _stream()),
            "attention_decode_tma")
     if num_splits > 1 and merge_counters is None:
         counters.own += 1  # the merge kernel
@@ -1221,7 +1392,7 @@ def attention_decode_tma(q, k_cache, v_cache, out, part_acc, part_ml, positions,
 
 def attention_prefill_mma(q, k_cache, v_cache, out, cu_q, pos0, block_table, entry0: int, n_entries: int,
                           max_new: int, window: int, scale: float, status=None, chunk: int = 0, sink=None,
-                          gate=None) -> None:
+                          gate=None, keep: int = 0) -> None:
     """Causal attention of the new tokens of the step's requests entry0 .. entry0 + n_entries - 1 over their
     pages, on tensor cores (bfloat16, head size 64 or 128).  cu_q [B + 1] gives each request's first token
     row, pos0 [B] the position of that token; max_new is the most new tokens any of them has.  ``chunk``,
@@ -1235,7 +1406,7 @@ def attention_prefill_mma(q, k_cache, v_cache, out, cu_q, pos0, block_table, ent
     _check(lib().ccb_attention_prefill_mma(_p(q), _p(k_cache), _p(v_cache), _p(out), _p(cu_q), _p(pos0),
                                               _p(block_table), block_table.stride(0), entry0, n_entries, max_new,
                                               nq, nkv, hd, page_size, num_pages, int(window), float(scale),
-                                              *_attn_extra(T, nq, q.dtype, chunk, sink, gate), _p(status),
+                                              *_attn_extra(T, nq, q.dtype, chunk, sink, gate, keep), _p(status),
                                               _stream()), "attention_prefill_mma")
 
 
@@ -1243,7 +1414,7 @@ def attention_decode_tma_fused(qkv, k_cache, v_cache, out, part_acc, part_ml, po
                                block_table, n_entries: int, row0: int, n_rows: int, nq: int, window: int,
                                scale: float, num_splits: int, q_norm_w, k_norm_w, eps: float, inv_freq,
                                write_kv: bool = True, status=None, merge_counters=None, bias=None,
-                               q_temperature=None, chunk: int = 0, sink=None, gate=None) -> None:
+                               q_temperature=None, chunk: int = 0, sink=None, gate=None, keep: int = 0) -> None:
     """attention_decode_tma for rows of ONE new token each, straight from the q|k|v product ``qkv``
     [T, (nq + 2 nkv) * hd] (only the nq query heads when ``write_kv`` is false): the kernel norms and rotates
     the queries itself and, with ``write_kv``, also the row's key, which it writes with the value to their
@@ -1273,7 +1444,7 @@ def attention_decode_tma_fused(qkv, k_cache, v_cache, out, part_acc, part_ml, po
         num_pages, int(window), float(scale), num_splits, _p(q_norm_w), _p(k_norm_w), float(eps), _p(inv_freq),
         1 if write_kv else 0, _p(bias), float(q_temperature[0]) if q_temperature else 0.0,
         int(q_temperature[1]) if q_temperature else 0, _p(merge_counters),
-        *_attn_extra(T, nq, qkv.dtype, chunk, sink, gate), _p(status), _stream()), "attention_decode_tma_fused")
+        *_attn_extra(T, nq, qkv.dtype, chunk, sink, gate, keep), _p(status), _stream()), "attention_decode_tma_fused")
     if num_splits > 1 and merge_counters is None:
         counters.own += 1  # the merge kernel
 
@@ -1284,7 +1455,7 @@ def attention_prefill_tc_fits(hd: int, page_size: int) -> bool:
 
 def attention_prefill_tc(q, k_cache, v_cache, out, cu_q, pos0, block_table, entry0: int, n_entries: int,
                          max_new: int, window: int, scale: float, status=None, chunk: int = 0, sink=None,
-                         gate=None) -> None:
+                         gate=None, keep: int = 0) -> None:
     """As attention_prefill_mma, with both products on tcgen05 tensor cores and the accumulators in tensor
     memory (128-token query tiles, TMA loads page by page).  Page size a power of two from 8 to 128.  Where the
     groups hold an even number of q heads, two heads of a group share a block and its key and value tiles."""
@@ -1297,7 +1468,7 @@ def attention_prefill_tc(q, k_cache, v_cache, out, cu_q, pos0, block_table, entr
     _check(lib().ccb_attention_prefill_tc(_p(q), _p(k_cache), _p(v_cache), _p(out), _p(cu_q), _p(pos0),
                                           _p(block_table), block_table.stride(0), entry0, n_entries, max_new, T,
                                           nq, nkv, hd, page_size, num_pages, int(window), float(scale),
-                                          *_attn_extra(T, nq, q.dtype, chunk, sink, gate), _p(status), _stream()),
+                                          *_attn_extra(T, nq, q.dtype, chunk, sink, gate, keep), _p(status), _stream()),
            "attention_prefill_tc")
 
 

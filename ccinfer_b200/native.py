@@ -32,7 +32,8 @@ ERRORS = {1: InvalidArgument, 2: KVBlockExhausted, 3: KVBlockDoubleFree, 4: KVIn
 
 
 class Group(Structure):
-    _fields_ = [("window", c_int), ("page_size", c_int), ("num_pages", c_int), ("chunk", c_int)]
+    _fields_ = [("window", c_int), ("page_size", c_int), ("num_pages", c_int), ("chunk", c_int),
+                ("keep_first", c_int)]
 
 
 class Options(Structure):
@@ -172,10 +173,10 @@ class HostCore:
     """One engine of the host core.  Sequences are named by 64-bit integers."""
 
     def __init__(self, groups, max_seqs: int, max_tokens_per_step: int, max_context: int):
-        """``groups``: (window or None, page_size, num_pages[, chunk or None]) per cache group."""
+        """``groups``: (window or None, page_size, num_pages[, chunk or None[, keep_first]]) per cache group."""
         self._lib = lib()
         self.n_groups = len(groups)
-        arr = (Group * max(1, self.n_groups))(*[Group(int(g[0] or 0), int(g[1]), int(g[2]), int(g[3] or 0) if len(g) > 3 else 0)
+        arr = (Group * max(1, self.n_groups))(*[Group(int(g[0] or 0), int(g[1]), int(g[2]), *(int(x or 0) for x in g[3:]))
                                                   for g in groups])
         opt = Options(self.n_groups, arr, int(max_seqs), int(max_tokens_per_step), int(max_context))
         self._h = c_void_p()

@@ -4,17 +4,18 @@ from .base import (Block, CachedTensor, CacheNeed, FeedForward, Mixer, Norm, Par
 from .block import LayerScaleBlock, PostNormBlock, PreNormBlock, SandwichNormBlock
 from .delta import ChannelGatedDelta
 from .embedding import LoopInput, OutputHead, TokenEmbedding, TokenSideInput
-from .feedforward import ClampedGLU, SquaredReLU, SwiGLU
+from .feedforward import ClampedGLU, GeluGLU, SquaredReLU, SwiGLU
 from .latent import LatentAttention
 from .linear_attention import GatedLinearAttention
+from .matrix_memory import ExponentialGateMemory, Retention
 from .moe import MixtureOfExperts
-from .norm import RMSNorm, StreamRows
+from .norm import LayerNorm, RMSNorm, StreamRows
 from .parallel import ParallelMixers
 from .position import NoPosition, QueryTemperature, RotaryHalf
 from .ssm import SelectiveStateSpace
 
-__all__ = ["Block", "CachedTensor", "CacheNeed", "ChannelGatedDelta", "ClampedGLU", "FeedForward",
-           "GatedLinearAttention", "GroupedQueryAttention", "LatentAttention", "LayerScaleBlock", "LoopInput", "Mixer",
+__all__ = ["Block", "CachedTensor", "CacheNeed", "ChannelGatedDelta", "ClampedGLU", "ExponentialGateMemory",
+           "FeedForward", "GatedLinearAttention", "GeluGLU", "GroupedQueryAttention", "LatentAttention", "LayerNorm", "LayerScaleBlock", "LoopInput", "Mixer",
            "MixtureOfExperts", "NoPosition", "Norm", "OutputHead", "ParallelMixers", "Part", "PositionEncoding",
-           "PostNormBlock", "PreNormBlock", "QueryTemperature", "RMSNorm", "Residual", "RotaryHalf", "SandwichNormBlock", "SelectiveStateSpace",
+           "PostNormBlock", "PreNormBlock", "QueryTemperature", "RMSNorm", "Residual", "Retention", "RotaryHalf", "SandwichNormBlock", "SelectiveStateSpace",
            "SquaredReLU", "StateNeed", "StreamRows", "SwiGLU", "TensorSpec", "TokenEmbedding", "TokenSideInput"]

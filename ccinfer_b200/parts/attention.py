@@ -40,7 +40,16 @@ merged projection); heads that talk to each other before the softmax (names
 ``talk`` [heads, heads] and optionally ``temp`` [heads]): head h's score is
 sum_g talk[h, g] * temp[g] * scale * (q_g . k), which one kernel computes for
 all heads of a query together (``csrc/attention_talking.cu``); a position
-encoding with an amplitude on its rotation (``PositionEncoding.amplitude``).
+encoding with an amplitude on its rotation (``PositionEncoding.amplitude``);
+the first tokens of a sequence kept visible behind a window (``keep_first``); a
+sink of a constant score (``sink_score``: one more term exp(score) in every
+softmax denominator, without a key or a value); keys that are the values as well
+(``keys_as_values``): there is no v projection, v is k as it leaves the
+convolution, before norm and rotation, and the norms of q and k run over all
+rows of their projection at once (weights of that size), which one kernel does
+from the product's rows to the cache (``csrc/qk_rows.cu``).  A permutation of
+the heads' coordinates then permutes the values too, and the output
+projection's columns with them.
 """
 from __future__ import annotations
 
@@ -60,7 +69,7 @@ class GroupedQueryAttention(Mixer):
     @property
     def kernel_groups(self):
         groups = ["talking"] if self.talking else ["attention"]
-        if self.taps or self.value_mix is not None:
+        if self.taps or self.value_mix is not None or self.keys_as_values:
             groups.append("recurrent")   # (the short convolutions live there)
         return tuple(groups)
 
@@ -68,7 +77,8 @@ class GroupedQueryAttention(Mixer):
                  position: PositionEncoding, names: dict, qk_norm_eps: Optional[float] = None,
                  window: Optional[int] = None, own_kv: bool = True, scale: Optional[float] = None,
                  value_dim: Optional[int] = None, float_weights: bool = False, chunk: Optional[int] = None,
-                 conv_taps: int = 0, value_mix: Optional[tuple] = None):
+                 conv_taps: int = 0, value_mix: Optional[tuple] = None, keep_first: int = 0,
+                 sink_score: Optional[float] = None, keys_as_values: bool = False):
         """``names``: tensor names under the keys q, k, v, o and (with qk_norm_eps) q_norm, k_norm; with
         q_bias, k_bias, v_bias the projections have biases; ``sink`` [heads]; ``gate`` [heads, hidden]; with
         ``conv_taps`` > 0 q_conv, k_conv, v_conv ([channels, taps]).  ``value_mix``: ("first", key) — this
@@ -102,18 +112,31 @@ class GroupedQueryAttention(Mixer):
             raise Unsupported("a layer that reads another layer's keys has no convolution, value mixing or gate")
         if (self.taps or self.value_mix) and self.has_bias:
             raise Unsupported("biases together with a convolution or value mixing")
+        self.keep_first = int(keep_first) if window is not None or self.chunk else 0   # (without a mask all are kept)
+        if self.keep_first < 0:
+            raise Unsupported("keep_first must be >= 0")
+        self.sink_score = None if sink_score is None else float(sink_score)
+        if self.sink_score is not None and "sink" in self.names:
+            raise Unsupported("a learned sink together with one of a constant score")
+        self.keys_as_values = bool(keys_as_values)
+        if self.keys_as_values and (self.qk_dim != self.v_dim or not own_kv or self.has_bias or value_mix is not None
+                                    or "gate" in self.names or "talk" in self.names):
+            raise Unsupported("keys that are the values: equal head sizes, keys of its own, no biases, value mixing, gate "
+                              "or talking heads")
         # attention beyond keys and values (every attention kernel takes them)
-        self.extras = bool(self.chunk or "sink" in self.names or "gate" in self.names)
+        self.extras = bool(self.chunk or self.keep_first or self.sink_score is not None or "sink" in self.names
+                           or "gate" in self.names)
         self.talking = "talk" in self.names
         if "temp" in self.names and not self.talking:
             raise Unsupported("a temperature per head comes with the heads' mixing matrix ('talk')")
-        if self.talking and self.chunk:
-            raise Unsupported("heads that talk to each other together with a chunked mask")
+        if self.talking and (self.chunk or self.keep_first or self.sink_score is not None):
+            raise Unsupported("heads that talk to each other together with a chunked mask, kept tokens or a constant sink")
         self.mix = None
         self.float_weights = bool(float_weights)
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(self.qk_dim)
         self.q_width, self.kv_width = self.nq * self.hd, self.nkv * self.hd
-        self.conv_width = self.q_width + 2 * self.kv_width      # the columns a convolution runs over: q | k | v
+        # the columns a convolution runs over: q | k | v, or q | k where the keys are the values
+        self.conv_width = self.q_width + (1 if self.keys_as_values else 2) * self.kv_width
         self.gate_off = self.conv_width                         # the gate's columns come after them
         self.in_width = self.conv_width + (-(-self.nq // 8) * 8 if "gate" in self.names else 0)
         self.bias = self.sink = self.conv_w = self.vmix = None
@@ -130,20 +153,24 @@ class GroupedQueryAttention(Mixer):
         n, D = self.names, self.hidden
         specs = [TensorSpec(n["q"], (self.nq * self.qk_dim, D)), TensorSpec(n["o"], (D, self.nq * self.v_dim))]
         if self.own_kv:
-            specs += [TensorSpec(n["k"], (self.nkv * self.qk_dim, D)), TensorSpec(n["v"], (self.nkv * self.v_dim, D))]
+            specs.append(TensorSpec(n["k"], (self.nkv * self.qk_dim, D)))
+            if not self.keys_as_values:
+                specs.append(TensorSpec(n["v"], (self.nkv * self.v_dim, D)))
         if self.has_bias:
             specs.append(TensorSpec(n["q_bias"], (self.nq * self.qk_dim,), role="vector"))
             if self.own_kv:
                 specs += [TensorSpec(n["k_bias"], (self.nkv * self.qk_dim,), role="vector"),
                           TensorSpec(n["v_bias"], (self.nkv * self.v_dim,), role="vector")]
         if self.qk_norm_eps is not None:
-            specs.append(TensorSpec(n["q_norm"], (self.qk_dim,), role="vector", init="one_plus_normal"))
+            nq, nkv = (self.nq, self.nkv) if self.keys_as_values else (1, 1)   # heads a weight covers
+            specs.append(TensorSpec(n["q_norm"], (nq * self.qk_dim,), role="vector", init="one_plus_normal"))
             if self.own_kv:
-                specs.append(TensorSpec(n["k_norm"], (self.qk_dim,), role="vector", init="one_plus_normal"))
+                specs.append(TensorSpec(n["k_norm"], (nkv * self.qk_dim,), role="vector", init="one_plus_normal"))
         if self.taps:
             specs += [TensorSpec(n["q_conv"], (self.nq * self.qk_dim, self.taps), role="vector"),
-                      TensorSpec(n["k_conv"], (self.nkv * self.qk_dim, self.taps), role="vector"),
-                      TensorSpec(n["v_conv"], (self.nkv * self.v_dim, self.taps), role="vector")]
+                      TensorSpec(n["k_conv"], (self.nkv * self.qk_dim, self.taps), role="vector")]
+            if not self.keys_as_values:
+                specs.append(TensorSpec(n["v_conv"], (self.nkv * self.v_dim, self.taps), role="vector"))
         if "sink" in n:
             specs.append(TensorSpec(n["sink"], (self.nq,), role="vector"))
         if "gate" in n:
@@ -157,10 +184,11 @@ class GroupedQueryAttention(Mixer):
         return specs
 
     def cache_need(self):
-        return CacheNeed.keys_and_values(self.nkv, self.hd, self.window, chunk=self.chunk or None)
+        return CacheNeed.keys_and_values(self.nkv, self.hd, self.window, chunk=self.chunk or None,
+                                         keep_first=self.keep_first)
 
     def state_need(self):
-        if self.taps > 1:   # the last taps - 1 rows of the q | k | v projection
+        if self.taps > 1:   # the last taps - 1 rows of the projection's convolved columns
             return StateNeed((self.taps - 1, self.conv_width), dtype=None, name="conv")
         return None
 
@@ -205,7 +233,9 @@ class GroupedQueryAttention(Mixer):
             return heads(laid_out(fetch(n[name]), n_heads, self.qk_dim), n_heads)
 
         if self.own_kv:
-            mats = [qk("q", self.nq), qk("k", self.nkv), laid_out(fetch(n["v"]), self.nkv, self.v_dim)]
+            mats = [qk("q", self.nq), qk("k", self.nkv)]
+            if not self.keys_as_values:
+                mats.append(laid_out(fetch(n["v"]), self.nkv, self.v_dim))
             if "gate" in n:
                 gate = torch.zeros((self.in_width - self.conv_width, self.hidden), dtype=mats[0].dtype, device=rt.device)
                 gate[:self.nq] = fetch(n["gate"])
@@ -221,9 +251,14 @@ class GroupedQueryAttention(Mixer):
         w_o = fetch(n["o"])
         if self.v_dim != hd:   # zero columns where the heads of o carry the added coordinates
             w_o = laid_out(w_o.t().contiguous(), self.nq, self.v_dim).t().contiguous()
+        if self.keys_as_values and idx is not None:   # the values' coordinates are permuted as the keys' are
+            w_o = heads(w_o.t().contiguous(), self.nq).t().contiguous()
         self.w_o = w_o
         self.norm_eps = self.qk_norm_eps
-        if self.qk_norm_eps is not None:
+        if self.qk_norm_eps is not None and self.keys_as_values:
+            self.q_norm_w, self.k_norm_w = (qk(name, heads_of).float().reshape(-1).contiguous()
+                                            for name, heads_of in (("q_norm", self.nq), ("k_norm", self.nkv)))
+        elif self.qk_norm_eps is not None:
             def norm_w(name):
                 w = fetch(n[name]).float()
                 if self.qk_dim != hd:
@@ -237,7 +272,7 @@ class GroupedQueryAttention(Mixer):
         amp = self.position.amplitude()
         if amp is not None:
             # a factor on cosine and sine is a factor on the rotated coordinate: it rides on the norms' weights
-            if self.qk_norm_eps is None:
+            if self.qk_norm_eps is None or self.keys_as_values:
                 raise Unsupported("a rotation with an amplitude needs the head norms whose weights carry it")
             amp = torch.from_numpy(amp).to(rt.device)
             self.q_norm_w = (self.q_norm_w * amp).contiguous()
@@ -253,8 +288,12 @@ class GroupedQueryAttention(Mixer):
             self.mix = (mix * self.scale).float().contiguous()
         if self.taps:
             # tap-major for the kernel: [taps, q | k | v channels]
-            self.conv_w = torch.cat([qk("q_conv", self.nq), qk("k_conv", self.nkv),
-                                     laid_out(fetch(n["v_conv"]), self.nkv, self.v_dim)], dim=0).float().t().contiguous()
+            convs = [qk("q_conv", self.nq), qk("k_conv", self.nkv)]
+            if not self.keys_as_values:
+                convs.append(laid_out(fetch(n["v_conv"]), self.nkv, self.v_dim))
+            self.conv_w = torch.cat(convs, dim=0).float().t().contiguous()
+        if self.sink_score is not None:
+            self.sink = torch.full((self.nq,), self.sink_score, dtype=torch.float32, device=rt.device)
         if "sink" in n:
             self.sink = fetch(n["sink"]).float().contiguous()
         if self.value_mix is not None and self.value_mix[0] == "mix":
@@ -292,7 +331,7 @@ class GroupedQueryAttention(Mixer):
                                               gate=gate, status=rt.status)
             return
         mma = rt.dtype == torch.bfloat16 and self.hd in kernels.DECODE_MMA_HEAD_SIZES and not self.float_weights
-        extra = {"chunk": self.chunk, "sink": self.sink, "gate": gate} if self.extras else {}
+        extra = {"chunk": self.chunk, "sink": self.sink, "gate": gate, "keep": self.keep_first} if self.extras else {}
         n_rows = step.n_single if mma else T
         if n_rows > 0:
             per_block = kernels.DECODE_MMA_HEADS_PER_BLOCK if mma else 0
@@ -324,7 +363,7 @@ class GroupedQueryAttention(Mixer):
         """A step of single tokens only, on the path of the TMA decode kernel (bfloat16, head size 64 or 128,
         a page size it takes), with few enough rows that every block redoing the queries' norm and rotation
         costs less than a kernel of its own."""
-        return (not self.float_weights and not self.talking and (self.bias is None or self.own_kv)
+        return (not self.float_weights and not self.talking and not self.keys_as_values and (self.bias is None or self.own_kv)
                 and self.rt.dtype == torch.bfloat16 and self.hd in kernels.DECODE_MMA_HEAD_SIZES
                 and kernels.attention_decode_tma_fits(self.hd, g.page_size)
                 and step.n_single == step.n_entries == step.n_tokens
@@ -359,10 +398,21 @@ class GroupedQueryAttention(Mixer):
         rt.linear(qkv, x, self.w_qkv)
         g = cache.group
         gate = qkv[:, self.gate_off:self.gate_off + self.nq] if "gate" in self.names else None
-        if self.taps or self.value_mix is not None:
+        if not self.keys_as_values and (self.taps or self.value_mix is not None):
             qkv = self._convolve(qkv, step, state, T)
         o = rt.scratch.get("attn_o", (rt.max_tokens, self.nq, self.hd), rt.dtype)[:T]
-        if self._fused_decode(step, g):
+        if self.keys_as_values:
+            q = rt.scratch.get("attn_q", (rt.max_tokens, self.nq, self.hd), rt.dtype)[:T]
+            taps = max(self.taps, 1)
+            kernels.qk_rows(qkv, q, cache.k, cache.v, self.conv_w, taps, state, self.q_norm_w, self.k_norm_w,
+                            self.norm_eps if self.norm_eps is not None else 1.0, self.qk_dim,
+                            self.position.rotary_table(), step.positions, g.slot_map, step.entry_of_token, step.cu_q,
+                            step.state_slot, step.n_entries, status=rt.status)
+            if taps > 1 and step.n_entries > step.n_single:
+                kernels.conv_state_rows(qkv, taps, self.conv_width, state, step.cu_q, step.state_slot, step.n_single,
+                                        step.n_entries - step.n_single)
+            self._attend(q, o, cache, step, T)
+        elif self._fused_decode(step, g):
             # every row brings one token: the decode attention norms and rotates the queries itself, writes
             # the row's key and value to their page and attends to them: one kernel less in every layer
             splits, n_acc, n_ml = kernels.attention_split_plan(T, self.nq, self.nkv, self.hd,
@@ -375,7 +425,7 @@ class GroupedQueryAttention(Mixer):
                 self.position.rotary_table(), write_kv=self.own_kv, status=rt.status,
                 merge_counters=rt.merge_counters if splits >= self.MERGE_IN_KERNEL_MIN_SPLITS else None,
                 bias=self.bias, q_temperature=self.position.query_temperature(), chunk=self.chunk, sink=self.sink,
-                gate=gate)
+                gate=gate, keep=self.keep_first)
         else:
             q = rt.scratch.get("attn_q", (rt.max_tokens, self.nq, self.hd), rt.dtype)[:T]
             args = (qkv, q, cache.k if self.own_kv else None, cache.v if self.own_kv else None, step.positions,

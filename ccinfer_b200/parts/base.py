@@ -75,23 +75,29 @@ class CacheNeed:
     pages wholly before that are given back while the request runs.  ``chunk``
     C: a query at position p reads the tokens from floor(p / C) * C on (runs of
     C positions counted from the sequence's start); pages wholly before the run
-    of the next token are given back.  Layers with equal (window, chunk) share a
+    of the next token are given back.  ``keep_first`` K (beside a window or a
+    chunk): every query also reads the first K tokens; their pages live as long
+    as the request.  Layers with equal (window, chunk, keep_first) share a
     page pool and block tables (a cache group); each layer has its own tensors
     of its own geometry.
     """
     tensors: Tuple[CachedTensor, ...]
     window: Optional[int] = None
     chunk: Optional[int] = None
+    keep_first: int = 0
 
     @classmethod
     def keys_and_values(cls, kv_heads: int, head_dim: int, window: Optional[int] = None,
-                        chunk: Optional[int] = None) -> "CacheNeed":
+                        chunk: Optional[int] = None, keep_first: int = 0) -> "CacheNeed":
         """Keys "k" and values "v" of an attention layer: [pages, kv_heads, page_size, head_dim] each."""
         shape = (int(kv_heads), int(head_dim))
-        return cls((CachedTensor("k", shape, token_axis=1), CachedTensor("v", shape, token_axis=1)), window, chunk)
+        return cls((CachedTensor("k", shape, token_axis=1), CachedTensor("v", shape, token_axis=1)), window, chunk,
+                   int(keep_first) if window is not None or chunk is not None else 0)
 
     @property
     def group_key(self):
+        if self.keep_first:
+            return ("kept", self.keep_first, self.window, self.chunk)
         if self.chunk is not None:
             return ("chunk", self.chunk) if self.window is None else ("window+chunk", self.window, self.chunk)
         return ("window", self.window) if self.window is not None else ("all",)
@@ -174,6 +180,19 @@ class UnscaledRows:
 
     def finish(self):
         return self._finish()
+
+
+class NormedPair:
+    """The output of a pair of mixers whose sum is still to be made: ca * unit(a) * wa + cb * unit(b) * wb, unit(x) =
+    x / sqrt(mean(x^2) + eps).  A block that sums it into the stream with ``kernels.norm_chain`` makes it there;
+    ``finish()`` returns it as a plain tensor (``Runtime.rows`` calls it)."""
+
+    def __init__(self, a, b, wa, wb, ca: float, cb: float, eps: float, finish):
+        self.a, self.args, self._finish = a, (b, wa, wb, float(ca), float(cb), float(eps)), finish
+        self.shape = a.shape
+
+    def finish(self):
+        return self._finish(self)
 
 
 class ResidualSink:

@@ -16,7 +16,7 @@ from typing import Optional
 import torch
 
 from .. import kernels
-from .base import Block, FeedForward, Mixer, Norm, Residual, ResidualSink
+from .base import Block, FeedForward, Mixer, Norm, NormedPair, Residual, ResidualSink
 
 
 def _groups_of(parts):
@@ -103,25 +103,28 @@ class PreNormBlock(Block):
 
 
 class SandwichNormBlock(Block):
-    """A norm before AND after each sublayer, the normed output scaled by a constant before the sum:
+    """A norm before AND after each sublayer, the normed output scaled by a constant before the sum, and optionally,
+    last, a token side input:
 
-        h += mult * post1(Mixer(norm1(h)));   h += mult * post2(FeedForward(norm2(h)))
+        h += mult * post1(Mixer(norm1(h)));   h += mult * post2(FeedForward(norm2(h)));   h += side(h, token)
 
-    The feed-forward (with norm2 and post2) may be absent.  All four are RMS norms with the same eps.  The
-    sum, the norm of the sublayer's output and the norm that reads the stream next are one kernel
-    (``kernels.postnorm_residual``): it also takes the rows that a repeated pass adds to the stream
-    (``Residual.next_add``) and leaves the next block's first norm as ``stream.ready``."""
+    The feed-forward (with norm2 and post2) may be absent.  The norms are RMS norms or layer norms.  The sum, the norm
+    of the sublayer's output and what reads the stream next are one kernel (``kernels.postnorm_residual`` where all
+    are RMS norms, else ``kernels.norm_chain``, which also makes the sum of a pair of mixers' normed outputs,
+    ``NormedPair``): it takes the rows that a repeated pass adds to the stream (``Residual.next_add``) and leaves the
+    next block's first norm as ``stream.ready``, or before a side input the stream's own rows for its gate."""
 
     def __init__(self, norm1, mixer: Mixer, post1, norm2=None, ffn: Optional[FeedForward] = None, post2=None,
-                 mult: float = 1.0):
+                 mult: float = 1.0, side=None):
         if (ffn is None) != (norm2 is None) or (ffn is None) != (post2 is None):
             raise ValueError("a feed-forward comes with its two norms, or none of the three is given")
         self.norm1, self.mixer, self.post1, self.norm2, self.ffn, self.post2 = norm1, mixer, post1, norm2, ffn, post2
-        self.mult = float(mult)
+        self.mult, self.side = float(mult), side
         self.rt = None
 
     def _parts(self):
-        return [p for p in (self.norm1, self.mixer, self.post1, self.norm2, self.ffn, self.post2) if p is not None]
+        return [p for p in (self.norm1, self.mixer, self.post1, self.norm2, self.ffn, self.post2, self.side)
+                if p is not None]
 
     @property
     def graph_safe(self):
@@ -138,36 +141,52 @@ class SandwichNormBlock(Block):
         self.rt = rt
         for p in self._parts():
             p.bind(rt, fetch)
+        self._side_spec = kernels.NormSpec("rms", self.side.w, None, self.side.eps) if self.side is not None else None
 
     @property
     def first_norm(self):
         return self.norm1
 
-    def _sum(self, stream: Residual, delta, post, nxt, last: bool):
-        """h += mult * post(delta) (+ the rows a repeated pass adds, after the block's last sum); with
-        ``nxt`` its rows are returned."""
+    def _sum(self, stream: Residual, delta, post, mult: float, nxt, last: bool, rows: bool = False):
+        """h += mult * post(delta) (+ the rows a repeated pass adds, after the block's last sum); returns the rows of
+        ``nxt`` (None where it is no norm that can be written ahead), or with ``rows`` the stream's own."""
         rt = self.rt
+        T, D = stream.h.shape
         add = None
         if last and stream.next_add is not None:
             add, stream.next_add = stream.next_add, None
+        nspec = nxt.spec() if nxt is not None and not rows and hasattr(nxt, "spec") else None
         y = None
-        usable = nxt is not None and hasattr(nxt, "w") and hasattr(nxt, "eps")
-        if usable:
-            y = rt.scratch.get(nxt.scratch_key, (rt.max_tokens, nxt.dim), rt.dtype)[:stream.h.shape[0]]
-        kernels.postnorm_residual(stream.h, rt.rows(delta), post.w, self.mult, post.eps, add=add,
-                                  y=y, w_next=nxt.w if usable else None, eps_next=nxt.eps if usable else 0.0)
+        if rows or nspec is not None:
+            key = "stream_rows" if rows else nxt.scratch_key
+            y = rt.scratch.get(key, (rt.max_tokens, D), rt.dtype)[:T]
+        if isinstance(delta, NormedPair):
+            kernels.norm_chain(stream.h, delta.a, post, nspec, y=y, mult=mult, add=add, pair=delta.args, status=rt.status)
+            return y
+        delta = rt.rows(delta)
+        if post.kind == "rms" and (nspec is None or nspec.kind == "rms"):
+            kernels.postnorm_residual(stream.h, delta, post.weight, mult, post.eps, add=add, y=y,
+                                      w_next=nspec.weight if nspec is not None else None,
+                                      eps_next=nspec.eps if nspec is not None else 0.0)
+        else:
+            kernels.norm_chain(stream.h, delta, post, nspec, y=y, mult=mult, add=add, status=rt.status)
         return y
 
     def forward(self, stream: Residual, step, cache, state) -> None:
         after = stream.next_norm
+        side = self.side is not None
         stream.takes_unscaled = False
         x = self.norm1.fold(stream)
         step.residual_sink = None
         a = self.mixer.forward(x, step, cache, state)
-        x = self._sum(stream, a, self.post1, self.norm2 if self.ffn is not None else after, self.ffn is None)
+        end = self.ffn is None
+        x = self._sum(stream, a, self.post1.spec(), self.mult, after if end else self.norm2, end and not side,
+                      rows=end and side)
         if self.ffn is not None:
             m = self.ffn.forward(x, step)
-            x = self._sum(stream, m, self.post2, after, True)
+            x = self._sum(stream, m, self.post2.spec(), self.mult, after, not side, rows=side)
+        if side:
+            x = self._sum(stream, self.side.forward(x, step), self._side_spec, 1.0, after, True)
         stream.ready = (after, x) if (after is not None and x is not None) else None
 
 

@@ -17,7 +17,7 @@ from .base import FeedForward, TensorSpec
 
 class SwiGLU(FeedForward):
     takes_unscaled = True
-    activation = None   # silu(gate) * up; a subclass names another one (see Runtime.gated_up)
+    activation = None   # silu(gate) * up; a subclass names another one (a kernels.GluAct, see Runtime.gated_up)
 
     def __init__(self, hidden: int, intermediate: int, names: dict):
         """``names``: tensor names under the keys gate, up, down."""
@@ -58,7 +58,13 @@ class ClampedGLU(SwiGLU):
     def __init__(self, hidden: int, intermediate: int, names: dict, limit: float, alpha: float = 1.702,
                  shift: float = 1.0):
         super().__init__(hidden, intermediate, names)
-        self.activation = ("clamped_glu", float(limit), float(alpha), float(shift))
+        self.activation = kernels.GluAct.clamped(limit, alpha, shift)
+
+
+class GeluGLU(SwiGLU):
+    """The same two products with gelu in its tanh form as the gate: m = (gelu(x Wg^T) * (x Wu^T)) Wd^T."""
+
+    activation = kernels.GluAct.gelu_tanh()
 
 
 class SquaredReLU(FeedForward):

@@ -5,8 +5,11 @@
     best choice score can be chosen; the ``top`` largest c are chosen; their weights are their s, as they are
     m = sum_chosen s_e * Wdown_e act(Wup_e x)  +  Wdown_s act(Wup_s x)      (a shared expert for every token)
 
-``activation`` "relu2": act(u) = relu(u)^2.  No biases.  ``activation`` "swiglu": every expert (the shared one
-too) has a gate matrix beside its up matrix, act = silu(Wgate_e x) * (Wup_e x).  ``rule`` (``kernels.RouteRule``)
+``activation`` "relu2": act(u) = relu(u)^2.  No biases.  ``activation`` "swiglu", or a ``kernels.GluAct``: every
+expert (the shared one too) has a gate matrix beside its up matrix, act = silu(Wgate_e x) * (Wup_e x), or that gated
+activation.  ``weight_on_input`` (gated experts): a token's weight for an expert multiplies what the expert reads
+instead of what it gives, expert(s_e x): its gate and up rows are linear in x, so the weight is applied to their
+results, in float, before the activation.  ``rule`` (``kernels.RouteRule``)
 says how logits become scores and weights (sigmoid scores, a group's score as the sum of its two best, chosen
 scores renormalised, a last factor); ``names["shared_gate"]``: the shared expert's result is multiplied by
 sigmoid(w_sg . x), one number per token (the row rides along as one more row of the router's matrix).
@@ -45,13 +48,21 @@ class MixtureOfExperts(FeedForward):
     TC_MIN_ROWS_PER_EXPERT = 8
 
     def __init__(self, hidden: int, experts: int, top: int, expert_ff: int, names: dict, groups: int = 1,
-                 keep: int = 1, shared_ff: int = 0, activation: str = "relu2", sparse=None, rule=None):
+                 keep: int = 1, shared_ff: int = 0, activation="relu2", sparse=None, rule=None,
+                 weight_on_input: bool = False):
         """``names``: "router", "correction" (optional), "up" and "down" (and "gate" with "swiglu") with ``{e}`` for
         the expert's number, "shared_up" / "shared_down" (/ "shared_gate_proj") with ``shared_ff`` > 0,
         "shared_gate" (optional)."""
-        if activation not in ("relu2", "swiglu"):
+        custom = isinstance(activation, kernels.GluAct)
+        if not custom and activation not in ("relu2", "swiglu"):
             raise Unsupported(f"expert activation {activation!r}")
-        self.glu = activation == "swiglu"
+        self.glu = custom or activation == "swiglu"
+        self.glu_act = activation if custom else None     # None: silu(gate) * up
+        self.weight_on_input = bool(weight_on_input)
+        if self.weight_on_input and not self.glu:
+            raise Unsupported("a weight on the experts' input comes with gated experts")
+        if custom and shared_ff and names.get("shared_gate"):
+            raise Unsupported("a gate on the shared expert together with an activation of its own")
         self.rule = rule
         if experts % groups or not (0 < keep <= groups) or not (0 < top <= (experts // groups) * keep):
             raise Unsupported(f"{experts} experts in {groups} groups of which {keep} are kept cannot give {top}")
@@ -182,20 +193,22 @@ class MixtureOfExperts(FeedForward):
         # the first product's rows an expert and its mode: with gates, gate and up rows in turn and the gated
         # activation as the epilogue
         F1, first = (2 * F, 2) if self.glu else (F, 0)
+        act_args = {"glu": self.glu_act, "weight_in": self.weight_on_input}
         if tc:
             xs = rt.scratch.get(f"moe_x_sorted:{top}", (max_pairs, D), rt.dtype)[:pairs]
             kernels.moe_gather_rows(xs, x, src_row)
-            kernels.moe_grouped_tc(act, xs, self.w_up, row_w, *tiles, F1, D, F1, first, status=rt.status)
+            kernels.moe_grouped_tc(act, xs, self.w_up, row_w, *tiles, F1, D, F1, first, status=rt.status, **act_args)
             kernels.moe_grouped_tc(rows, act, self.w_down, row_w, *tiles, D, F, F, 1, status=rt.status)
         else:
-            kernels.moe_grouped(act, x, src_row, self.w_up, F1 * self.w_up.stride(0), row_w, *tiles, F1, D, BM, first)
+            kernels.moe_grouped(act, x, src_row, self.w_up, F1 * self.w_up.stride(0), row_w, *tiles, F1, D, BM, first,
+                                **act_args)
             kernels.moe_grouped(rows, act, None, self.w_down, F, row_w, *tiles, D, F, BM, 1)
         shared = None
         if self.SF and self.glu:
             sa = rt.scratch.get(f"moe_shared_act:{self.SF}", (rt.max_tokens, self.SF), rt.dtype)[:T]
             gu = rt.scratch.get(f"moe_shared_gate_up:{self.SF}", (rt.max_tokens, 2 * self.SF), rt.dtype)[:T]
             rt.linear(gu, x, self.w_shared_up)
-            kernels.moe_dense_glu_act(sa, gu, None, 0, 1, self.SF, self._shared_gate(T))
+            kernels.moe_dense_glu_act(sa, gu, None, 0, 1, self.SF, self._shared_gate(T), glu=self.glu_act)
             shared = rt.scratch.get("moe_shared_out", (rt.max_tokens, D), rt.dtype)[:T]
             rt.linear(shared, sa, self.w_shared_down)
         elif self.SF:
@@ -219,7 +232,8 @@ class MixtureOfExperts(FeedForward):
         if self.glu:
             gu = rt.scratch.get("moe_gate_up", (rt.max_tokens, 2 * self.width), rt.dtype)[:T]
             rt.linear(gu, x, self.w_up)
-            kernels.moe_dense_glu_act(act, gu, dense, self.E, self.F, self.SF, self._shared_gate(T))
+            kernels.moe_dense_glu_act(act, gu, dense, self.E, self.F, self.SF, self._shared_gate(T), glu=self.glu_act,
+                                      weight_in=self.weight_on_input)
         else:
             rt.linear(act, x, self.w_up)
             kernels.moe_dense_act(act, dense, self.E, self.F, self.SF)

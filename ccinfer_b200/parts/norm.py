@@ -1,4 +1,4 @@
-"""RMSNorm: y = x * rsqrt(mean(x^2) + eps) * w (7QiC/ccInfer: src/kernel/norm/rms_norm.cu:24-60)."""
+"""Norms.  RMSNorm: y = x * rsqrt(mean(x^2) + eps) * w (7QiC/ccInfer: src/kernel/norm/rms_norm.cu:24-60)."""
 from __future__ import annotations
 
 import torch
@@ -36,6 +36,10 @@ class RMSNorm(Norm):
             self.w = (self.w.float() + self.weight_offset).contiguous()
         if self.weight_scale != 1.0:
             self.w = (self.w.float() * self.weight_scale).contiguous()
+
+    def spec(self):
+        """This norm as ``kernels.norm_chain`` takes it."""
+        return kernels.NormSpec("rms", self.w, None, self.eps)
 
     def fold(self, stream: Residual, rows=None, n_rows=None):
         rt = self.rt
@@ -86,6 +90,53 @@ class RMSNorm(Norm):
     def apply(self, x):
         y = torch.empty_like(x)  # the part alone, outside a step: not a buffer of the pool
         kernels.rmsnorm(y, x, self.w, self.eps)
+        return y
+
+
+class LayerNorm(Norm):
+    """y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias, over the stream's float rows
+    (``kernels.norm_chain``).  (Its weights are not called ``w``: a part that looks for an RMS norm's weight to fold
+    into a kernel of its own does not find one here.)"""
+
+    def __init__(self, dim: int, eps: float, weight_name: str, bias_name: str, scratch_key: str = "normed"):
+        self.dim, self.eps, self.scratch_key = int(dim), float(eps), scratch_key
+        self.weight_name, self.bias_name = weight_name, bias_name
+        self.weight = self.bias = None
+        self.rt = None
+
+    def tensor_specs(self):
+        return [TensorSpec(self.weight_name, (self.dim,), role="vector", init="one_plus_normal"),
+                TensorSpec(self.bias_name, (self.dim,), role="vector")]
+
+    def bind(self, rt, fetch):
+        self.rt = rt
+        self.weight = fetch(self.weight_name).float().contiguous()
+        self.bias = fetch(self.bias_name).float().contiguous()
+
+    def spec(self):
+        return kernels.NormSpec("layer", self.weight, self.bias, self.eps)
+
+    def fold(self, stream: Residual, rows=None, n_rows=None):
+        rt = self.rt
+        T = stream.h.shape[0]
+        ready, stream.ready = stream.ready, None
+        stream.unscaled = None
+        if ready is not None and rows is None and ready[0] is self and stream.pending is None:
+            return ready[1]
+        delta = None if stream.pending is None else rt.rows(stream.pending)
+        if rows is None:
+            y = rt.scratch.get(self.scratch_key, (rt.max_tokens, self.dim), rt.dtype)[:T]
+            kernels.norm_chain(stream.h, delta, nxt=self.spec(), y=y, status=rt.status)
+            stream.pending = None
+        else:
+            n = rows.numel() if n_rows is None else n_rows
+            y = rt.scratch.get(self.scratch_key + "_rows", (rt.max_tokens, self.dim), rt.dtype)[:n]
+            kernels.norm_chain(stream.h, delta, nxt=self.spec(), y=y, row_idx=rows, n_rows=n, status=rt.status)
+        return y
+
+    def apply(self, x):
+        y = torch.empty_like(x)
+        kernels.norm_chain(x.float().contiguous(), nxt=self.spec(), y=y, status=self.rt.status)
         return y
 
 

@@ -40,7 +40,8 @@ class RotaryHalf(PositionEncoding):
     """
 
     def __init__(self, head_dim: int, theta: float, rotary_dim: int = None, interleaved: bool = False,
-                 linear_scaling: float = None, query_temperature=None, ramp_scaling: dict = None):
+                 linear_scaling: float = None, query_temperature=None, ramp_scaling: dict = None,
+                 wavelength_scaling: dict = None):
         """``linear_scaling`` s: every frequency is divided by s (positions are stretched by s); the table is
         then evaluated in float64 and rounded once.  ``query_temperature``: see ``QueryTemperature``.
         ``ramp_scaling`` {"factor", "original", "fast", "slow"}: only the slow pairs are stretched.  A pair that
@@ -50,7 +51,10 @@ class RotaryHalf(PositionEncoding):
         divided by ``factor``; between the two bounds the share b of the divided frequency grows linearly from 0 to
         1 (the bounds are kept at least 0.001 apart), freq = b * f / factor + (1 - b) * f.  Cosine and sine both
         carry the factor 1 + log(factor) / 10 (``amplitude``; the attention mixer puts it into the weights of its
-        head norms)."""
+        head norms).
+        ``wavelength_scaling`` {"factor", "low", "high", "original"}: a pair of frequency f has the wavelength 2 pi / f.
+        Below original / high it keeps its frequency, above original / low it has it divided by ``factor``, and
+        between the two, with s = (original / wavelength - low) / (high - low), it gets (1 - s) f / factor + s f."""
         rotary_dim = int(head_dim if rotary_dim is None else rotary_dim)
         self.ramp_scaling = None
         if ramp_scaling is not None:
@@ -60,6 +64,13 @@ class RotaryHalf(PositionEncoding):
             if not (self.ramp_scaling["factor"] > 0 and self.ramp_scaling["original"] > 0
                     and self.ramp_scaling["fast"] > 0 and self.ramp_scaling["slow"] > 0):
                 raise ValueError("ramp_scaling: factor, original, fast and slow must be > 0")
+        self.wavelength_scaling = None
+        if wavelength_scaling is not None:
+            if linear_scaling is not None or ramp_scaling is not None:
+                raise ValueError("one kind of frequency scaling at a time")
+            sc = self.wavelength_scaling = {k: float(wavelength_scaling[k]) for k in ("factor", "low", "high", "original")}
+            if not (sc["factor"] > 0 and sc["original"] > 0 and 0 < sc["low"] <= sc["high"]):
+                raise ValueError("wavelength_scaling: factor and original > 0, 0 < low <= high")
         if linear_scaling is not None and not (linear_scaling > 0):
             raise ValueError("linear_scaling must be > 0")
         self.linear_scaling = None if linear_scaling is None else float(linear_scaling)
@@ -75,6 +86,8 @@ class RotaryHalf(PositionEncoding):
         table = np.zeros(self.head_dim // 2, dtype=np.float32)
         if self.ramp_scaling is not None:
             table[:self.rotary_dim // 2] = self.ramp_frequencies().astype(np.float32)
+        elif self.wavelength_scaling is not None:
+            table[:self.rotary_dim // 2] = self.wavelength_frequencies().astype(np.float32)
         elif self.linear_scaling is None:
             table[:self.rotary_dim // 2] = rotary_inv_freq(self.rotary_dim, self.theta)
         else:
@@ -99,6 +112,17 @@ class RotaryHalf(PositionEncoding):
         hi = min(math.ceil(where(sc["slow"])), dims - 1)
         ramp = np.clip((np.arange(dims // 2, dtype=np.float64) - lo) / max(hi - lo, 0.001), 0.0, 1.0)
         return f / sc["factor"] * ramp + f * (1.0 - ramp)
+
+    def wavelength_frequencies(self) -> np.ndarray:
+        """float64 [rotary_dim / 2]: the frequencies under ``wavelength_scaling``."""
+        sc = self.wavelength_scaling
+        f = np.power(np.float64(self.theta), -2.0 * np.arange(self.rotary_dim // 2, dtype=np.float64) / self.rotary_dim)
+        wavelength = 2.0 * np.pi / f
+        span = sc["high"] - sc["low"]
+        s = (sc["original"] / wavelength - sc["low"]) / (span if span > 0 else 1.0)
+        mixed = (1.0 - s) * f / sc["factor"] + s * f
+        return np.where(wavelength < sc["original"] / sc["high"], f,
+                        np.where(wavelength > sc["original"] / sc["low"], f / sc["factor"], mixed))
 
     def amplitude(self):
         """None, or float32 [head_dim] in the kernels' layout: the factor on cosine and sine of each coordinate's

@@ -159,7 +159,7 @@ def test_clamped_glu_as_the_epilogue_of_the_product(kind, M, F, K):
     wu = (torch.randn(F, K, generator=g) * 2.0 / K ** 0.5).to(torch.bfloat16)
     w = kernels.interleave_gate_up(wg.cuda(), wu.cuda(), kernels.SWIGLU_BLOCK)
     act = torch.empty(M, F, dtype=torch.bfloat16, device="cuda")
-    kernels.gemm_glu_bf16(act, x.cuda(), w, 1.5, 1.702, 1.0, kind)
+    kernels.gemm_glu_bf16(act, x.cuda(), w, kernels.GluAct.clamped(1.5, 1.702, 1.0), kind)
     want = plain.clamped_glu(x.double() @ wg.double().T, x.double() @ wu.double().T, 1.5)
     assert (act.cpu().double() - want).abs().max() < 2e-2 * max(1.0, want.abs().max())
 
