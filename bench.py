@@ -35,10 +35,10 @@ runs one of the two other workloads of the reference's benchmark record through 
 continuous batch at the Qwen3-14B shape; four 16,384-token prompts at the Qwen3-32B shape) and prints a
 line of its own: output tokens a second, the distribution of the step calls, the pages' high water.
 
-    python bench.py --design tugelorn|dufizen|burolorn|gevovik [--design-sizes mid,8b] [--layers L] [--design-profile]
+    python bench.py --design tugelorn|dufizen|burolorn|gevovik|duzizen [--design-sizes mid,8b] [--layers L] [--design-profile]
 
 measures another design of the package beside its closest model (Tugelorn beside Qwen3, Dufizen beside
-Tugelorn, Burolorn beside Qwen3, Gevovik beside Tugelorn) at equal layer sizes (same width, heads, head size,
+Tugelorn, Burolorn beside Qwen3, Gevovik beside Tugelorn, Duzizen beside Dufizen) at equal layer sizes (same width, heads, head size,
 intermediate size, vocabulary and number of layers; random weights): one prompt of 2,048 and of 8,192 tokens
 in steps of 2,048 (tokens a second) and decode steps of 1 and 8 requests after 2,048-token prompts, replayed
 from CUDA graphs (tokens a second), one JSON line per size.  With --design-profile it only runs a prompt and a
@@ -371,6 +371,31 @@ def gevovik_config(size: str, layers: int):
     return GevovikConfig.from_json(j)
 
 
+def duzizen_config(size: str, layers: int):
+    """Layers in turn: a pair of attention whose values are its keys (four taps on q and k, norms over the whole
+    projections, half of each head rotated with stretched long wavelengths, a window of 1,024 beside which the first
+    four tokens stay, one added to the denominator) beside a retention of half as many heads, and an exponentially gated
+    matrix memory of H heads; the feed-forward in turn dense (F) and a mixture of 32 gated experts of F / 4 of which
+    4 are used (F intermediate channels per token either way); layer norms before and after every sublayer, a token
+    side input of 256 columns, an embedding with a pair table."""
+    from ccinfer_b200.config.duzizen import DuzizenConfig
+    D, H, G, hd, F, V = DESIGN_SIZES[size]
+    pair = {"type": "parallel", "mixer": {
+        "left": {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "conv": 4,
+                 "mask": {"size": 1024, "keep_first": 4},
+                 "rot": {"dims": hd // 2, "base": 500000.0,
+                         "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+        "right": {"heads": H // 2, "dim": hd, "vdim": hd, "decay": [1 - 2.0 ** -(5 + i / 4) for i in range(H // 2)],
+                  "rot": {"dims": hd, "base": 10000.0}}}}
+    memory = {"type": "mlstm", "mixer": {"heads": H, "dim": hd, "vdim": hd, "gate_cap": 15.0}}
+    mlps = [{"kind": "dense", "ff": F},
+            {"kind": "moe", "expert": {"ff": F // 4, "limit": 7.0}, "router": {"experts": 32, "top": 4}}]
+    j = {"architecture": "Duzizen", "vocab": V, "width": D, "norm": {"eps": 1e-5}, "token_side": {"dim": 256},
+         "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}},
+         "layers": [dict((pair, memory)[i % 2], mlp=mlps[(i // 2 + i) % 2]) for i in range(layers)]}
+    return DuzizenConfig.from_json(j)
+
+
 def run_design(args) -> int:
     import numpy as np
     import torch
@@ -380,7 +405,8 @@ def run_design(args) -> int:
 
     # design -> (its configuration at a size, the closest model it is measured beside)
     designs = {"tugelorn": (tugelorn_config, "qwen3"), "dufizen": (dufizen_config, "tugelorn"),
-               "burolorn": (burolorn_config, "qwen3"), "gevovik": (gevovik_config, "tugelorn")}
+               "burolorn": (burolorn_config, "qwen3"), "gevovik": (gevovik_config, "tugelorn"),
+               "duzizen": (duzizen_config, "dufizen")}
     if args.design not in designs:
         print(json.dumps({"error": f"unknown design {args.design!r}"}))
         return 2
@@ -498,7 +524,7 @@ def main() -> int:
     ap.add_argument("--shape", default="8b", choices=["8b", "14b", "32b"], help="layer shape of --profile-steps")
     ap.add_argument("--workload", default="decode", choices=["decode", "mix14b", "long32b"],
                     help="decode (the default line) or one of the two other workloads of the benchmark record")
-    ap.add_argument("--design", default=None, help="tugelorn (beside Qwen3), dufizen (beside Tugelorn), burolorn (beside Qwen3) or gevovik (beside Tugelorn): that design beside its closest model at "
+    ap.add_argument("--design", default=None, help="tugelorn (beside Qwen3), dufizen (beside Tugelorn), burolorn (beside Qwen3), gevovik (beside Tugelorn) or duzizen (beside Dufizen): that design beside its closest model at "
                                                    "equal layer sizes")
     ap.add_argument("--design-sizes", default="mid,8b", help="layer sizes of --design: " + ", ".join(DESIGN_SIZES))
     ap.add_argument("--design-profile", action="store_true", help="with --design: a prompt and four eager decode steps")
