@@ -65,6 +65,7 @@ GROUPS = {
         "short_conv.cu",
         "qk_rows.cu",
         "scalar_memory.cu",
+        "memory_chunks.cu",
         "delta_rule.cu",
         "linear_attention.cu",
         "ssm.cu",

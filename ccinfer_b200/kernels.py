@@ -184,7 +184,13 @@ _SIGNATURES = {
                    + [c_int] * 9 + [c_void_p, c_void_p],
     "ccb_memory_prepare": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                            c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p],
-    "ccb_memory_gates": [c_void_p, c_int, c_void_p, c_void_p, c_float] + [c_void_p] * 6 + [c_int] * 3 + [c_void_p],
+    "ccb_memory_gates": [c_void_p, c_int, c_void_p, c_void_p, c_float] + [c_void_p] * 6 + [c_int] * 5 + [c_void_p],
+    "ccb_memory_rotate_split": [c_void_p, c_int, c_int, c_int, c_void_p, c_int] + [c_void_p] * 5
+                               + [c_int, c_int, c_int, c_float, c_float, c_void_p],
+    "ccb_memory_step": [c_void_p] + [c_int] * 5 + [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_float]
+                       + [c_void_p] * 4 + [c_int] + [c_void_p] * 4 + [c_float, c_float, c_int, c_void_p]
+                       + [c_int] * 7 + [c_float, c_float, c_int, c_int, c_void_p],
+    "ccb_memory_chunks": [c_void_p] * 4 + [c_int, c_void_p, c_int] + [c_void_p] * 6 + [c_int] * 7 + [c_float, c_void_p],
     "ccb_memory_output": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int,
                           c_float, c_int, c_void_p],
     "ccb_relu_squared": [c_void_p, c_void_p, c_longlong, c_int, c_void_p],
@@ -1019,23 +1025,94 @@ def memory_prepare(proj, offsets, inv_freq, rot_dims: int, positions, qn, kn, vv
                                     _stream()), "memory_prepare")
 
 
-def memory_gates(z, bias_i, bias_f, cap: float, m_state, cu_q, state_slot, decay, put, floor, n_entries: int,
-                 H: int) -> None:
-    """The exponential gates of a matrix memory with their running maximum (``scalar_memory.cu``): ``z`` float [T, 2 H]
-    pre-activations (input gates, forget gates); ``m_state`` float [slots, H] is moved on; decay, put and floor float
-    [T, H] are exp(f + m_before - m), exp(i - m) and exp(-m)."""
+def memory_rotate_split(proj, offsets, inv_freq, rot_dims: int, positions, q, k, H: int, dk: int, q_mult: float,
+                        k_mult: float) -> None:
+    """As ``memory_prepare`` for q and k alone, each left as two bfloat16, its rounding and what that left: ``q`` and
+    ``k`` are pairs of [T, H dk] tensors.  dk and rot_dims are multiples of 4."""
+    _cuda(inv_freq, positions, *q, *k)
+    T = q[0].shape[0]
+    assert proj.dtype == torch.bfloat16 and proj.stride(1) == 1 and proj.shape[0] == T
+    assert all(x.dtype == torch.bfloat16 and x.shape == (T, H * dk) for x in (*q, *k))
+    _check(lib().ccb_memory_rotate_split(_p(proj), proj.stride(0), offsets[0], offsets[1], _p(inv_freq), int(rot_dims),
+                                         _p(positions), _p(q[0]), _p(q[1]), _p(k[0]), _p(k[1]), T, H, dk, float(q_mult),
+                                         float(k_mult), _stream()), "memory_rotate_split")
+
+
+def memory_gates(z, bias_i, bias_f, cap: float, m_state, cu_q, state_slot, decay, put, floor, n_entries: int, H: int,
+                 entry0: int = 0, logs: bool = False) -> None:
+    """The exponential gates of a matrix memory with their running maximum (``scalar_memory.cu``) for the entries
+    entry0 .. entry0 + n_entries - 1: ``z`` float [T, 2 H] pre-activations (input gates, forget gates); ``m_state``
+    float [slots, H] is moved on; decay, put and floor float [T, H] are exp(f + m_before - m), exp(i - m) (their
+    logarithms with ``logs``) and exp(-m)."""
     _cuda(bias_i, bias_f, m_state, cu_q, state_slot, decay, put, floor)
     assert z.dtype == torch.float32 and z.stride(1) == 1 and z.shape[1] >= 2 * H and m_state.dtype == torch.float32
     assert decay.shape == put.shape == floor.shape == (z.shape[0], H) and decay.dtype == torch.float32
     _check(lib().ccb_memory_gates(_p(z), z.stride(0), _p(bias_i), _p(bias_f), float(cap), _p(m_state), _p(cu_q),
-                                  _p(state_slot), _p(decay), _p(put), _p(floor), int(n_entries), H, m_state.shape[0],
-                                  _stream()), "memory_gates")
+                                  _p(state_slot), _p(decay), _p(put), _p(floor), int(entry0), int(n_entries), H,
+                                  m_state.shape[0], 1 if logs else 0, _stream()), "memory_gates")
+
+
+def memory_step(y, proj, offsets, gates, state, inv_freq, rot_dims: int, positions, cu_q, state_slot, n_entries: int, H: int,
+                dk: int, dv: int, q_mult: float, k_mult: float, eps: float, weight=None, den_eps: float = 0.0,
+                silu_gate: bool = False, ones: bool = False) -> None:
+    """One token of each of the first ``n_entries`` entries through a matrix memory, from the projection's row to the
+    gated, normed output y [T, H dv]: ``memory_prepare``, the gates, the recurrence and ``memory_output`` in one kernel.
+
+    ``offsets``: columns of q, k, v and the output gate in ``proj``.  ``gates``: a float [H] of constant decays, or
+    (z, column of the input gates, of the forget gates, bias_i, bias_f, cap, m_state) with ``z`` a float view of rows."""
+    _cuda(y, state, inv_freq, positions, cu_q, state_slot, weight)
+    assert proj.is_cuda and proj.stride(1) == 1 and proj.shape[0] == y.shape[0] and y.shape[1] == H * dv
+    assert state.dtype == torch.float32 and tuple(state.shape[1:]) == (H, dv + (1 if ones else 0), dk)
+    oq, ok, ov, og = offsets
+    assert max(oq + H * dk, ok + H * dk, ov + H * dv, og + H * dv) <= proj.shape[1]
+    z = bi = bf = m_state = decay = None
+    zi = zf = ldz = 0
+    cap = 1.0
+    if isinstance(gates, tuple):
+        z, zi, zf, bi, bf, cap, m_state = gates
+        assert z.dtype == torch.float32 and z.stride(1) == 1 and max(zi, zf) + H <= z.shape[1]
+        ldz = z.stride(0)
+    else:
+        decay = gates
+        assert decay.dtype == torch.float32 and decay.numel() == H and not ones
+    _check(lib().ccb_memory_step(_p(proj), proj.stride(0), oq, ok, ov, og, _p(z), ldz, int(zi), int(zf), _p(bi), _p(bf),
+                                 float(cap), _p(m_state), _p(decay), _p(state), _p(inv_freq), int(rot_dims), _p(positions),
+                                 _p(cu_q), _p(state_slot), _p(weight), float(eps), float(den_eps), 1 if silu_gate else 0,
+                                 _p(y), y.stride(0), int(n_entries), H, dk, dv, 1 if ones else 0, state.shape[0],
+                                 float(q_mult), float(k_mult), _dt(proj), _dt(y), _stream()), "memory_step")
+
+
+MEMORY_CHUNK = 64   # tokens the chunked form of the recurrence takes at a time
+
+
+def memory_chunks_fits(dtype, dk: int, dv: int) -> bool:
+    return dtype == torch.bfloat16 and dk in (64, 128) and dv % 16 == 0
+
+
+def memory_chunks(q, k, v, log_decay, log_put, state, out, cu_q, state_slot, entry0: int, n_entries: int, H: int, dk: int,
+                  dv: int, q_mult: float) -> None:
+    """The recurrence of ``memory_recurrence`` (its read-out times ``q_mult``) for the entries entry0 .. of a step, in
+    chunks of 64 tokens on tensor cores.  ``q`` and ``k``: pairs (bfloat16 rows [T, >= H dk], what their rounding left
+    or None); ``v`` bfloat16 rows [T, >= H dv]; ``log_decay`` and ``log_put`` (None: 0) float [T, H]; ``state`` float
+    [slots, H, dv (+ 1), dk] and ``out`` float [T, H, dv (+ 1)], the further value being always one."""
+    _cuda(log_decay, log_put, state, out, cu_q, state_slot)
+    dvo = out.shape[2]
+    rows = [x for x in (*q, *k) if x is not None]
+    assert all(x.dtype == torch.bfloat16 and x.stride(1) == 1 and x.stride(0) == rows[0].stride(0) for x in rows)
+    assert v.dtype == torch.bfloat16 and v.stride(1) == 1 and state.dtype == out.dtype == torch.float32
+    assert tuple(state.shape[1:]) == (H, dvo, dk) and log_decay.shape == (out.shape[0], H) and dvo - dv in (0, 1)
+    _check(lib().ccb_memory_chunks(_p(q[0]), _p(q[1]), _p(k[0]), _p(k[1]), rows[0].stride(0), _p(v), v.stride(0),
+                                   _p(log_decay), _p(log_put), _p(state), _p(out), _p(cu_q), _p(state_slot), int(entry0),
+                                   int(n_entries), H, dk, dv, dvo, state.shape[0], float(q_mult), _stream()),
+           "memory_chunks")
 
 
 def memory_recurrence(qn, kn, vv, decay, put, state, out, cu_q, state_slot, n_entries: int, H: int, dk: int,
-                      dv: int) -> None:
+                      dv: int, entry0: int = 0) -> None:
     """S <- a_t S + b_t k_t v_t^T, o_t = S^T q_t with one decay a_t (``decay`` float [T, H]) and one factor on the
-    write (``put`` float [T, H], None: 1) per head and token; S is ``state`` float [slots, H, dv, dk]."""
+    write (``put`` float [T, H], None: 1) per head and token; S is ``state`` float [slots, H, dv, dk].  Entries entry0
+    .. entry0 + n_entries - 1."""
+    cu_q, state_slot = cu_q[entry0:], state_slot[entry0:]
     _cuda(qn, kn, vv, decay, put, state, out, cu_q, state_slot)
     _check(lib().ccb_ssm_recurrence(_p(qn), _p(kn), _p(vv), _p(decay), _p(put), _p(state), _p(out), _p(cu_q),
                                     _p(state_slot), int(n_entries), H, H, dk, dv, _stream()), "memory_recurrence")
@@ -1049,7 +1126,7 @@ def memory_output(y, o, gate, H: int, dv: int, eps: float, weight=None, floor=No
     _cuda(y, o, weight, floor)
     T = y.shape[0]
     assert y.shape == (T, H * dv) and o.shape == (T, H, dv + (1 if floor is not None else 0)) and o.dtype == torch.float32
-    assert gate.dtype == y.dtype and gate.stride(1) == 1 and gate.shape[0] == T and gate.shape[1] >= H * dv
+    assert gate.is_cuda and gate.dtype == y.dtype and gate.stride(1) == 1 and gate.shape[0] == T and gate.shape[1] >= H * dv
     assert weight is None or (weight.dtype == torch.float32 and weight.numel() == H * dv)
     _check(lib().ccb_memory_output(_p(y), _p(o), _p(floor), float(den_eps), _p(gate), gate.stride(0),
                                    1 if silu_gate else 0, _p(weight), T, H, dv, float(eps), _dt(y), _stream()),

@@ -14,11 +14,18 @@ b_t = exp(i_t - m_t) never overflow.  The keys are summed by the same recurrence
 o_t = S^T q_t / (max(|n . q|, exp(-m_t)) + 1e-6); y = unit(o) * w * sigmoid(Wg x) with a weight per channel of all heads.
 n is one more value channel of S, whose value is always one: n . q is then one more column of the read-out.
 
-Both end with Wo.  q, k, v and the output gate are ONE merged product of x; the exponential gates' two rows per head
-are a product with a float result.  Everything after the products is float (``csrc/scalar_memory.cu``, and the plain
-form of the recurrence in ``csrc/delta_rule.cu``).
+Both end with Wo.  q, k, v and the output gate (and, where the step only brings a few single tokens, the exponential
+gates' two rows per head, which otherwise are a product with a float result of their own) are ONE merged product of x.
+Everything after the products is float:
+
+* requests that bring one token: one kernel from the projection's row to the gated output (``kernels.memory_step``);
+* portions of prompts, bfloat16, key sizes 64 and 128: chunks of 64 tokens on tensor cores (``csrc/memory_chunks.cu``),
+  then the normaliser, norm and gate;
+* everything else: float rows and the plain form of the recurrence in ``csrc/delta_rule.cu``.
 """
 from __future__ import annotations
+
+import math
 
 import torch
 
@@ -27,7 +34,8 @@ from ..errors import Unsupported
 from .base import Mixer, StateNeed, TensorSpec
 from .position import RotaryHalf
 
-DENOMINATOR_EPS = 1e-6   # added to the normaliser of the exponentially gated memory
+DENOMINATOR_EPS = 1e-6    # added to the normaliser of the exponentially gated memory
+LEAST_LOG_DECAY = -80.0   # a decay below e^-80 keeps nothing that a float can tell from zero
 
 
 def _pad8(n: int) -> int:
@@ -48,7 +56,8 @@ class ScalarDecayMemory(Mixer):
         self.oq, self.ok = 0, _pad8(qk)
         self.ov = self.ok + _pad8(qk)
         self.og = self.ov + _pad8(vw)
-        self.in_width = self.og + _pad8(vw)
+        self.in_width = self.og + _pad8(vw)        # q | k | v | g
+        self.full_width = self.in_width            # ... and what a subclass puts after them
         self.rt = None
 
     def tensor_specs(self):
@@ -60,22 +69,30 @@ class ScalarDecayMemory(Mixer):
     def _memory_need(self):
         return StateNeed((self.H, self.dv + self.ones, self.dk), torch.float32, "S")
 
+    # rows of the merged projection beyond q, k, v and g: (offset, tensor)
+    def _more_rows(self, fetch):
+        return []
+
     def bind(self, rt, fetch):
         self.rt = rt
         n = self.names
-        w = torch.zeros((self.in_width, self.hidden), dtype=rt.dtype, device=rt.device)
-        for off, name in ((self.oq, "q"), (self.ok, "k"), (self.ov, "v"), (self.og, "g")):
-            t = fetch(n[name])
+        w = torch.zeros((self.full_width, self.hidden), dtype=rt.dtype, device=rt.device)
+        for off, t in [(off, fetch(n[name])) for off, name in ((self.oq, "q"), (self.ok, "k"), (self.ov, "v"),
+                                                               (self.og, "g"))] + self._more_rows(fetch):
             w[off:off + t.shape[0]] = t
-        self.w_in = w
+        self.w_full, self.w_in, self.w_more = w, w[:self.in_width], w[self.in_width:]
         self.w_o = fetch(n["o"])
 
     # rotation and constant factors of the queries and keys: (inverse frequencies, dims, q factor, k factor)
     def _rotation(self):
         return None, 0, 1.0, 1.0
 
-    # a_t and b_t of the step's rows (b None: one), and exp(-m_t) (None: no normaliser)
-    def _gates(self, x, step, state, T):
+    # the gates of the portions' rows: a_t and b_t (b None: one), or their logarithms, and exp(-m_t) (None: no normaliser)
+    def _gates(self, z, step, state, T, logs: bool):
+        raise NotImplementedError
+
+    # the same for single tokens, as ``kernels.memory_step`` takes it
+    def _step_gates(self, z, state):
         raise NotImplementedError
 
     def forward(self, x, step, cache, state):
@@ -84,21 +101,57 @@ class ScalarDecayMemory(Mixer):
         T = x.shape[0]
         H, dk, dv, dvo = self.H, self.dk, self.dv, self.dv + self.ones
         f32 = torch.float32
-        proj = rt.scratch.get("memory_proj", (rt.max_tokens, self.in_width), rt.dtype)[:T]
-        rt.linear(proj, x, self.w_in)
-        decay, put, floor = self._gates(x, step, state, T)
+        # (layers of other sizes have buffers of their own: one that only long steps use must not grow once CUDA graphs
+        # hold the pool's addresses)
+        size = f":{H}:{dk}:{dvo}"
+        single, many = step.n_single, step.n_entries - step.n_single
+        z = None
+        if self.full_width > self.in_width and (rt.dtype == f32 or (many == 0 and T <= kernels.FEWROWS_MAX_ROWS)):
+            # a few single tokens: the product is a stream of the weights, and a float result costs nothing
+            proj = rt.scratch.get("memory_proj_full" + size, (rt.max_tokens if rt.dtype == f32 else kernels.FEWROWS_MAX_ROWS,
+                                                       self.full_width), f32)[:T]
+            rt.linear(proj, x, self.w_full)
+            z = proj[:, self.in_width:]
+        else:
+            proj = rt.scratch.get("memory_proj" + size, (rt.max_tokens, self.in_width), rt.dtype)[:T]
+            rt.linear(proj, x, self.w_in)
+            if self.full_width > self.in_width:
+                z = rt.scratch.get("memory_gate_z" + size, (rt.max_tokens, self.full_width - self.in_width), f32)[:T]
+                rt.linear(z, x, self.w_more)
         S = state["S"] if isinstance(state, dict) else state
-        qn = rt.scratch.get("delta_q", (rt.max_tokens, H, dk), f32)[:T]
-        kn = rt.scratch.get("delta_k", (rt.max_tokens, H, dk), f32)[:T]
-        vv = rt.scratch.get("delta_v", (rt.max_tokens, H, dvo), f32)[:T]
         inv_freq, rot_dims, q_mult, k_mult = self._rotation()
-        kernels.memory_prepare(proj, (self.oq, self.ok, self.ov), inv_freq, rot_dims, step.positions, qn, kn, vv, H, dk,
-                               dv, q_mult, k_mult, ones=bool(self.ones))
-        o = rt.scratch.get("delta_o", (rt.max_tokens, H, dvo), f32)[:T]
-        kernels.memory_recurrence(qn, kn, vv, decay, put, S, o, step.cu_q, step.state_slot, step.n_entries, H, dk, dvo)
+        den_eps = DENOMINATOR_EPS if self.ones else 0.0
         y = rt.scratch.get("delta_y", (rt.max_tokens, H * dv), rt.dtype)[:T]
-        kernels.memory_output(y, o, proj[:, self.og:], H, dv, self.eps, weight=self.norm_w, floor=floor,
-                              den_eps=DENOMINATOR_EPS if floor is not None else 0.0, silu_gate=self.silu_gate)
+        if single > 0:
+            kernels.memory_step(y, proj, (self.oq, self.ok, self.ov, self.og), self._step_gates(z, state), S, inv_freq,
+                                rot_dims, step.positions, step.cu_q, step.state_slot, single, H, dk, dv, q_mult, k_mult,
+                                self.eps, weight=self.norm_w, den_eps=den_eps, silu_gate=self.silu_gate,
+                                ones=bool(self.ones))
+        if many > 0:
+            chunks = kernels.memory_chunks_fits(rt.dtype, dk, dv) and rot_dims % 4 == 0
+            decay, put, floor = self._gates(z, step, state, T, chunks)
+            o = rt.scratch.get("delta_o" + size, (rt.max_tokens, H, dvo), f32)[:T]
+            if chunks:
+                v = proj[:, self.ov:]
+                if rot_dims or k_mult != 1.0:   # (float rows that are no longer bfloat16: as two bfloat16 each)
+                    halves = [rt.scratch.get(f"memory_split{i}{size}", (rt.max_tokens, H * dk), rt.dtype)[:T] for i in range(4)]
+                    q, k = halves[:2], halves[2:]
+                    kernels.memory_rotate_split(proj, (self.oq, self.ok), inv_freq, rot_dims, step.positions, q, k, H, dk,
+                                                1.0, k_mult)
+                else:
+                    q, k = (proj[:, self.oq:], None), (proj[:, self.ok:], None)
+                kernels.memory_chunks(q, k, v, decay, put, S, o, step.cu_q, step.state_slot, single, many, H, dk, dv, q_mult)
+            else:
+                qn = rt.scratch.get("delta_q" + size, (rt.max_tokens, H, dk), f32)[:T]
+                kn = rt.scratch.get("delta_k" + size, (rt.max_tokens, H, dk), f32)[:T]
+                vv = rt.scratch.get("delta_v" + size, (rt.max_tokens, H, dvo), f32)[:T]
+                kernels.memory_prepare(proj, (self.oq, self.ok, self.ov), inv_freq, rot_dims, step.positions, qn, kn, vv,
+                                       H, dk, dv, q_mult, k_mult, ones=bool(self.ones))
+                kernels.memory_recurrence(qn, kn, vv, decay, put, S, o, step.cu_q, step.state_slot, many, H, dk, dvo,
+                                          entry0=single)
+            kernels.memory_output(y[single:], o[single:], proj[single:, self.og:], H, dv, self.eps, weight=self.norm_w,
+                                  floor=floor[single:] if floor is not None else None, den_eps=den_eps,
+                                  silu_gate=self.silu_gate)
         out = rt.scratch.get(self.out_key, (rt.max_tokens, self.hidden), rt.dtype)[:T]
         return rt.linear(out, y, self.w_o)
 
@@ -126,7 +179,10 @@ class Retention(ScalarDecayMemory):
     def bind(self, rt, fetch):
         super().bind(rt, fetch)
         # the same decay for every token: rows that nobody writes again
-        self.decay_rows = torch.tensor(self.decay, dtype=torch.float32, device=rt.device).repeat(rt.max_tokens, 1)
+        self.decays = torch.tensor(self.decay, dtype=torch.float32, device=rt.device)
+        self.decay_rows = self.decays.repeat(rt.max_tokens, 1)
+        logs = [max(math.log(d), LEAST_LOG_DECAY) if d > 0 else LEAST_LOG_DECAY for d in self.decay]
+        self.log_rows = torch.tensor(logs, dtype=torch.float32, device=rt.device).repeat(rt.max_tokens, 1)
         self.inv_freq = None
         if self.rotation is not None:
             self.rotation.bind(rt, fetch)
@@ -135,8 +191,11 @@ class Retention(ScalarDecayMemory):
     def _rotation(self):
         return self.inv_freq, (self.rotation.rotary_dim if self.rotation is not None else 0), 1.0, self.dk ** -0.5
 
-    def _gates(self, x, step, state, T):
-        return self.decay_rows[:T], None, None
+    def _gates(self, z, step, state, T, logs):
+        return (self.log_rows if logs else self.decay_rows)[:T], None, None
+
+    def _step_gates(self, z, state):
+        return self.decays
 
 
 class ExponentialGateMemory(ScalarDecayMemory):
@@ -149,6 +208,7 @@ class ExponentialGateMemory(ScalarDecayMemory):
         if not gate_cap > 0:
             raise Unsupported("gate_cap must be > 0")
         self.cap = float(gate_cap)
+        self.full_width = self.in_width + _pad8(2 * self.H)   # the input gates' rows, then the forget gates'
 
     def tensor_specs(self):
         n, D = self.names, self.hidden
@@ -160,22 +220,25 @@ class ExponentialGateMemory(ScalarDecayMemory):
     def state_need(self):
         return [self._memory_need(), StateNeed((self.H,), torch.float32, "m")]
 
+    def _more_rows(self, fetch):
+        return [(self.in_width, fetch(self.names["i"])), (self.in_width + self.H, fetch(self.names["f"]))]
+
     def bind(self, rt, fetch):
         super().bind(rt, fetch)
         n = self.names
-        self.w_gates = torch.cat([fetch(n["i"]), fetch(n["f"])], dim=0).contiguous()
         self.i_bias, self.f_bias = fetch(n["i_bias"]).float().contiguous(), fetch(n["f_bias"]).float().contiguous()
         self.norm_w = fetch(n["norm"]).float().contiguous()
 
     def _rotation(self):
         return None, 0, self.dk ** -0.5, 1.0
 
-    def _gates(self, x, step, state, T):
+    def _gates(self, z, step, state, T, logs):
         rt, H = self.rt, self.H
-        z = rt.scratch.get("memory_gate_z", (rt.max_tokens, 2 * H), torch.float32)[:T]
-        rt.linear(z, x, self.w_gates)
-        decay, put, floor = (rt.scratch.get(key, (rt.max_tokens, H), torch.float32)[:T]
+        decay, put, floor = (rt.scratch.get(f"{key}:{H}", (rt.max_tokens, H), torch.float32)[:T]
                              for key in ("memory_decay", "memory_put", "memory_floor"))
         kernels.memory_gates(z, self.i_bias, self.f_bias, self.cap, state["m"], step.cu_q, step.state_slot, decay, put,
-                             floor, step.n_entries, H)
+                             floor, step.n_entries - step.n_single, H, entry0=step.n_single, logs=logs)
         return decay, put, floor
+
+    def _step_gates(self, z, state):
+        return (z, 0, self.H, self.i_bias, self.f_bias, self.cap, state["m"])

@@ -252,3 +252,192 @@ def generate(cfg, w, prompt, n):
 
 
 greedy = generate
+
+
+# ---- configurations of the tests and random weights -----------------------------------------------------------
+def memory(heads, dim, vdim, gate_cap):
+    return ("mlstm", {"heads": heads, "dim": dim, "vdim": vdim, "gate_cap": gate_cap})
+
+
+def attention(heads, kv_heads, dim, scale, conv=0, window=None, keep_first=0, rot=None, scaling=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": scale}
+    if conv:
+        m["conv"] = conv
+    if window is not None:
+        m["mask"] = {"size": window, "keep_first": keep_first}
+    if rot is not None:
+        m["rot"] = {"dims": rot[0], "base": rot[1]}
+        if scaling is not None:
+            m["rot"]["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+    return m
+
+
+def keep(heads, dim, vdim, decay, rot=None):
+    m = {"heads": heads, "dim": dim, "vdim": vdim, "decay": list(decay)}
+    if rot is not None:
+        m["rot"] = {"dims": rot[0], "base": rot[1]}
+    return m
+
+
+def pair(left, right):
+    return ("parallel", {"left": left, "right": right})
+
+
+def dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(n, top, ff, limit):
+    return {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": {"experts": n, "top": top}}
+
+
+def model(vocab, width, eps, layers, bigram=None, side=None):
+    """``layers``: [((type, mixer), mlp or None)]; ``bigram``: (buckets, mul_prev, mul_cur)."""
+    j = {"architecture": "Duzizen", "vocab": vocab, "width": width, "norm": {"eps": eps},
+         "layers": [{"type": t, "mixer": m, "mlp": q} for (t, m), q in layers]}
+    if bigram is not None:
+        j["embedding"] = {"bigram": dict(zip(("buckets", "mul_prev", "mul_cur"), bigram))}
+    if side is not None:
+        j["token_side"] = {"dim": side}
+    return j
+
+
+# name -> (configuration, page size)
+CONFIGS = {
+    # a window of 21 over pages of 8 with three kept tokens, part of each head rotated with stretched wavelengths;
+    # experts of which three are used; a layer without feed-forward
+    "A": (model(90, 64, 1e-5, [
+        (memory(3, 16, 24, 9.0), moe(6, 3, 24, 0.8)),
+        (pair(attention(4, 2, 16, 0.3, conv=3, window=21, keep_first=3, rot=(8, 5000.0), scaling=(4.0, 1.0, 3.0, 64)),
+              keep(2, 16, 8, (0.9, 0.997), rot=(16, 10000.0))), dense(72)),
+        (memory(2, 8, 16, 4.0), None),
+        (pair(attention(2, 1, 32, 0.2, conv=4, window=33, keep_first=9, rot=(32, 300.0)),
+              keep(3, 12, 20, (0.5, 0.98, 1.0), rot=(4, 100.0))), moe(5, 1, 16, 1.5))],
+        bigram=(61, 3, 11), side=10), 8),
+    # sizes that are multiples of nothing; one head; no convolution, no pair table, no side input, no mask (every
+    # earlier key), no rotation on the right
+    "B": (model(71, 44, 1e-6, [
+        (pair(attention(1, 1, 10, 0.4, rot=(6, 500.0)), keep(1, 6, 10, (0.95,))), dense(37)),
+        (memory(1, 7, 5, 15.0), dense(64)),
+        (pair(attention(3, 3, 20, 0.25, conv=1, window=1, keep_first=0), keep(2, 10, 6, (0.0, 0.9), rot=(2, 10.0))), None),
+        (memory(5, 4, 12, 2.0), moe(3, 2, 11, 0.5))]), 4),
+    # tensor-core head sizes, a kept token more than a page, a window shorter than a page, one that ends on a page
+    "C": (model(130, 96, 1e-5, [
+        (pair(attention(6, 2, 64, 0.125, conv=4, window=36, keep_first=17, rot=(32, 10000.0), scaling=(2.0, 1.0, 4.0, 32)),
+              keep(2, 64, 64, (0.96, 0.999), rot=(64, 10000.0))), moe(8, 2, 32, 2.0)),
+        (memory(2, 64, 64, 12.0), dense(128)),
+        (pair(attention(2, 2, 128, 0.09, conv=2, window=5, keep_first=1, rot=(128, 1000.0)),
+              keep(1, 128, 32, (0.99,), rot=(64, 500.0))), dense(64)),
+        (memory(1, 128, 96, 8.0), moe(4, 4, 40, 1.0))], bigram=(31, 1, 7), side=16), 16),
+}
+
+
+def config(name):
+    return CONFIGS[name]
+
+
+def tensor_shapes(cfg):
+    D, V = cfg["width"], cfg["vocab"]
+    s = {"embed": (V, D), "head": (V, D), "final.norm": (D,), "final.norm.b": (D,)}
+    b = (cfg.get("embedding") or {}).get("bigram")
+    if b is not None:
+        s["bigram"] = (b["buckets"] + 1, D)
+    side = cfg.get("token_side")
+    if side is not None:
+        s["side.embed"] = (V, side["dim"] * len(cfg["layers"]))
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if layer["mlp"] is not None else ()):
+            s[p + n] = s[p + n + ".b"] = (D,)
+        q = p + "mix."
+        if layer["type"] == "mlstm":
+            H, qk, vw = m["heads"], m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            s.update({q + "q": (qk, D), q + "k": (qk, D), q + "v": (vw, D), q + "g": (vw, D), q + "o": (D, vw),
+                      q + "norm": (vw,), q + "i": (H, D), q + "i.b": (H,), q + "f": (H, D), q + "f.b": (H,)})
+        else:
+            a, r = m["left"], m["right"]
+            qw, kw = a["heads"] * a["dim"], a["kv_heads"] * a["dim"]
+            s.update({q + "left.q": (qw, D), q + "left.k": (kw, D), q + "left.q.norm": (qw,), q + "left.k.norm": (kw,),
+                      q + "left.o": (D, qw), q + "left.out": (D,), q + "right.out": (D,)})
+            if a.get("conv"):
+                s.update({q + "left.q.conv": (qw, a["conv"]), q + "left.k.conv": (kw, a["conv"])})
+            qk, vw = r["heads"] * r["dim"], r["heads"] * r["vdim"]
+            s.update({q + "right.q": (qk, D), q + "right.k": (qk, D), q + "right.v": (vw, D), q + "right.g": (vw, D),
+                      q + "right.o": (D, vw)})
+        f = layer["mlp"]
+        if f is not None and f["kind"] == "dense":
+            s.update({p + "mlp.gate": (f["ff"], D), p + "mlp.up": (f["ff"], D), p + "mlp.down": (D, f["ff"])})
+        elif f is not None:
+            s[p + "mlp.router"] = (f["router"]["experts"], D)
+            for e in range(f["router"]["experts"]):
+                F = f["expert"]["ff"]
+                s.update({p + f"mlp.e{e}.gate": (F, D), p + f"mlp.e{e}.up": (F, D), p + f"mlp.e{e}.down": (D, F)})
+        if side is not None:
+            s.update({p + "side.gate": (side["dim"], D), p + "side.proj": (D, side["dim"]), p + "side.norm": (D,)})
+    return s
+
+
+def random_weights(cfg, seed, sharp=1.0):
+    """Random tensors (values that bfloat16 holds exactly).  Matrices N(0, 1 / fan-in); norm weights around one;
+    ``sharp`` multiplies the attention layers' query norms, so that the softmax sits on few keys; the routers' rows are
+    scaled up so that few choices are close."""
+    g = torch.Generator().manual_seed(seed)
+    w = {}
+    for name, shape in tensor_shapes(cfg).items():
+        leaf = name.split(".")[-1]
+        if leaf == "b":
+            t = 0.3 * torch.randn(shape, generator=g)
+            if name.endswith(".f.b"):
+                t = t + 3.0                      # remember for a while
+        elif name.endswith((".conv",)):
+            t = torch.randn(shape, generator=g) / math.sqrt(shape[1])
+        elif len(shape) == 1:
+            t = 1.0 + 0.2 * torch.randn(shape, generator=g)
+            if name.endswith("left.q.norm"):
+                t = t * sharp
+        elif name in ("embed", "bigram", "side.embed"):
+            t = torch.randn(shape, generator=g)
+        else:
+            t = torch.randn(shape, generator=g) / math.sqrt(shape[-1])
+            if leaf == "router":
+                t = t * 3.0
+        w[name] = t.to(torch.bfloat16).to(torch.float32)
+    return w
+
+
+def random_config(seed):
+    """A configuration drawn at random: (config, page size).  Every size, count, constant and option that a
+    configuration may state is drawn, the order of the layers too."""
+    import random
+    r = random.Random(seed)
+    width = r.choice([32, 40, 48, 64, 96])
+
+    def rot_of(dim, scaled):
+        dims = r.choice([d for d in (2, 4, 8, 16, 32, 64, dim // 2 * 2) if d <= dim])
+        scaling = (r.choice([1.5, 4.0, 8.0]), 1.0, r.choice([2.0, 4.0]), r.choice([16, 64, 512])) if scaled else None
+        return (dims, r.choice([100.0, 10000.0, 500000.0])), scaling
+
+    layers = []
+    for _ in range(r.randint(2, 5)):
+        if r.random() < 0.45:
+            mix = memory(r.choice([1, 2, 3, 4]), r.choice([4, 8, 16, 48, 64, 128]), r.choice([4, 8, 24, 32, 64, 96]),
+                         r.choice([1.0, 5.0, 12.0]))
+        else:
+            kv, dim = r.choice([1, 2, 4]), r.choice([6, 8, 16, 24, 32, 48, 64, 128])
+            rot, scaling = rot_of(dim, r.random() < 0.6) if r.random() < 0.85 else (None, None)
+            left = attention(kv * r.choice([1, 2, 3]), kv, dim, dim ** -0.5 * r.choice([0.7, 1.0, 1.6]), conv=r.randint(0, 5),
+                             window=r.choice([None, 1, 3, 7, 16, 33, 72]), keep_first=r.choice([0, 1, 4, 5, 16, 21]),
+                             rot=rot, scaling=scaling)
+            if "mask" not in left:
+                left.pop("keep_first", None)
+            H, d2 = r.choice([1, 2, 3]), r.choice([4, 8, 16, 48, 64, 128])
+            right = keep(H, d2, r.choice([4, 8, 24, 32, 64, 96]), [r.choice([0.2, 0.9, 0.98, 0.999, 1.0]) for _ in range(H)],
+                         rot=rot_of(d2, False)[0] if r.random() < 0.8 else None)
+            mix = pair(left, right)
+        n = r.choice([2, 4, 7, 16])
+        mlp = r.choice([None, dense(r.choice([16, 30, 64, 100])), moe(n, r.randint(1, min(n, 3)), r.choice([8, 20, 32, 64]),
+                                                                     r.choice([0.4, 1.0, 7.0]))])
+        layers.append((mix, mlp))
+    return model(r.randint(50, 200), width, r.choice([1e-5, 1e-6]), layers,
+                 bigram=(r.choice([7, 31, 97]), r.randint(1, 40), r.randint(1, 40)) if r.random() < 0.7 else None,
+                 side=r.choice([None, 3, 8, 24])), r.choice([4, 8, 16])
