@@ -798,15 +798,26 @@ FUZZ_SEEDS = int(os.environ.get("CCB_FUZZ_SEEDS", "12"))
 def test_random_configurations(tmp_path, seed):
     """Configurations drawn at random (sizes, head counts, the order of the layers, windows, kept tokens, taps,
     constants, with and without pair table, side input, rotation, scaling, mask and feed-forward): a mixed trace with a
-    pool that is just large enough, and every request whole, in both types.  A drawn model may have rows that magnify
-    rounding, so the 32-bit bound is 2e-4 here (a wrong mechanism moves the logits by their own size), and the bfloat16
-    runs, which are there for the kernels' paths at odd sizes, want finite rows, a median within 3e-2 and at most one
-    row in eight beyond 8e-2."""
+    pool that is just large enough, and every request whole, in both types.  A drawn model has rows that magnify
+    rounding (a side input of three columns is normalised whatever its size, a memory of four key channels may nearly
+    cancel), so the 32-bit bound of a row grows with how far that row moves in the plain implementation when every
+    weight is changed by a millionth; the bfloat16 runs, which are there for the kernels' paths at odd sizes, want
+    finite rows, a median within 3e-2, and beyond 8e-2 at most one row in eight, or half as many again as the plain
+    implementation moves that far when every weight is changed by half a bfloat16 step (choices of experts flip)."""
     cfg, page = plain.random_config(1000 + seed)
     d = str(tmp_path / "drawn")
     cfg, w = write_model(d, cfg=cfg, seed=seed, sharp=1.5)
     reqs = requests_of(cfg, [1, 2, page, page + 1, 35, 72, 74, 110], seed)
     ref = {rid: plain.forward(cfg, w, t).numpy() for rid, t in reqs.items()}
+    gen = torch.Generator().manual_seed(seed)
+    scale = {rid: max(1e-6, float(np.abs(r).max())) for rid, r in ref.items()}
+
+    def moves(by):   # per request: how far each row moves when every weight is changed by that share
+        moved = {k: v.double() * (1 + by * torch.randn(v.shape, dtype=torch.float64, generator=gen)) for k, v in w.items()}
+        return {rid: np.abs(plain.forward(cfg, moved, t).numpy() - ref[rid]).max(1) / scale[rid] for rid, t in reqs.items()}
+
+    bound = {rid: TOL32 + 10 * m for rid, m in moves(1e-6).items()}
+    far_rows = sum(int((m > TOL16).sum()) for m in moves(2e-3).values())
     for dtype in ("float32", "bfloat16"):
         for steps in (helpers.trace_mixed(reqs, max_live=4, seed=seed, portion_choices=(2, 3, 5, 17, 40)),
                       helpers.trace_whole(reqs)):
@@ -814,12 +825,14 @@ def test_random_configurations(tmp_path, seed):
             eng = engine_of(d, dtype, page, pool, max_requests=4, use_graphs=(dtype == "bfloat16"))
             rows = helpers.replay(eng, steps)
             if dtype == "float32":
-                helpers.compare(rows, ref, 2e-4, f"drawn configuration {seed}")
+                for (rid, pos), row in rows.items():
+                    err = float(np.abs(row - ref[rid][pos]).max()) / scale[rid]
+                    assert np.isfinite(row).all() and err <= bound[rid][pos], (seed, rid, pos, err, bound[rid][pos])
             else:
-                errs = np.array([np.abs(row - ref[rid][pos]).max() / max(1e-6, np.abs(ref[rid]).max())
-                                 for (rid, pos), row in rows.items()])
+                errs = np.array([np.abs(row - ref[rid][pos]).max() / scale[rid] for (rid, pos), row in rows.items()])
                 assert np.isfinite(errs).all() and np.median(errs) <= 3e-2, (seed, float(np.median(errs)))
-                assert int((errs > TOL16).sum()) <= len(errs) // 8, (seed, int((errs > TOL16).sum()), len(errs))
+                beyond = int((errs > TOL16).sum())
+                assert beyond <= max(len(errs) // 8, 3 * far_rows // 2), (seed, beyond, far_rows, len(errs))
             assert all(p.used_pages == 0 for p in eng.cache.pools)
 
 
@@ -947,6 +960,7 @@ def test_a_far_token_decides_through_the_state(tmp_path, which):
         else:
             w["l0.mix.left.out"] = torch.zeros_like(w["l0.mix.left.out"])
         w["l0.norm1"], w["l0.norm1.b"] = torch.ones(32), torch.zeros(32)
+        w["l0.norm1b"] = torch.full((32,), 3.0)       # the mixer outweighs the token's own row
         w["embed"][2:, :16] *= 0.05
         w["embed"][1, :16] = w["embed"][0, :16]
 
