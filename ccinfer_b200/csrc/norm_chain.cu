@@ -12,8 +12,8 @@
 // written to h, and y holds them in the order of row_idx.  The stream and every sum are float; delta and y are of
 // the storage type.
 //
-//   norm_chain_vec    D a multiple of 4 up to 8,192 with aligned rows: everything a row needs (weights too, up to
-//                     4,096) is asked for at once with 16-byte loads and stays in registers between the sums
+//   norm_chain_vec    D a multiple of 4 up to 8,192 with aligned rows: everything a row needs (with few rows the
+//                     weights too) is asked for at once with 16-byte loads and stays in registers between the sums
 //   norm_chain_row    any D whose row fits shared memory
 #include "common.cuh"
 
@@ -74,8 +74,9 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {
   return t;
 }
 
-// Normalises x[NV] (the row's pieces this thread holds) in place.
-template <int NV, int kThreads>
+// Normalises x[NV] (the row's pieces this thread holds) in place.  kHeld: the weights are in w and b; else they are
+// loaded where they are needed.
+template <int NV, int kThreads, bool kHeld>
 __device__ __forceinline__ void apply_stage(const NormStage& st, float4* x, const float4* w, const float4* b, int nvec,
                                             int D, float* red) {
   if (st.kind == 0) return;
@@ -99,22 +100,28 @@ __device__ __forceinline__ void apply_stage(const NormStage& st, float4* x, cons
 #pragma unroll
   for (int j = 0; j < NV; ++j)
     if (threadIdx.x + j * kThreads < nvec) {
-      x[j].x = x[j].x * inv * w[j].x; x[j].y = x[j].y * inv * w[j].y;
-      x[j].z = x[j].z * inv * w[j].z; x[j].w = x[j].w * inv * w[j].w;
-      if (st.kind == 2) { x[j].x += b[j].x; x[j].y += b[j].y; x[j].z += b[j].z; x[j].w += b[j].w; }
+      const int i = 4 * (threadIdx.x + j * kThreads);
+      const float4 wj = kHeld ? w[j] : V4<float>::load(st.w + i);
+      x[j].x = x[j].x * inv * wj.x; x[j].y = x[j].y * inv * wj.y;
+      x[j].z = x[j].z * inv * wj.z; x[j].w = x[j].w * inv * wj.w;
+      if (st.kind == 2) {
+        const float4 bj = kHeld ? b[j] : V4<float>::load(st.b + i);
+        x[j].x += bj.x; x[j].y += bj.y; x[j].z += bj.z; x[j].w += bj.w;
+      }
     }
 }
 
-template <typename T, int NV, int kThreads>
+// kAhead: the weights are asked for with the row (few rows: latency); else each when it is needed (many rows: fewer
+// registers, more blocks on an SM).
+template <typename T, int NV, int kThreads, bool kAhead, bool kPair>
 __global__ void __launch_bounds__(kThreads)
 norm_chain_vec_kernel(T* __restrict__ y, float* __restrict__ h, const T* __restrict__ delta, const NormPair pair,
                       const NormStage post, float mult, const float* __restrict__ add, const NormStage next,
                       const int* __restrict__ row_idx, int n_src_rows, int D, int* status) {
-  constexpr bool kAhead = NV <= 2;   // the weights are loaded with the row (registers)
   __shared__ float red[64];
   const int r = blockIdx.x;
   const int nvec = D >> 2;
-  float4 pw[NV], pb[NV], nw[NV], nb[NV], wa[NV], wb[NV];
+  float4 pw[NV], pb[NV], nw[NV], nb[NV];
   auto load_stage = [&](const NormStage& st, float4* w, float4* b) {
     if (st.kind == 0) return;
 #pragma unroll
@@ -150,17 +157,19 @@ norm_chain_vec_kernel(T* __restrict__ y, float* __restrict__ h, const T* __restr
       if (delta) d[j] = V4<T>::load(delta + (size_t)src * D + 4 * i);
     }
   }
-  if (pair.second != nullptr) {
+  if (kPair) {
     const T* br = static_cast<const T*>(pair.second) + (size_t)src * D;
-    float4 e[NV];
+    float4 e[NV], wa[NV], wb[NV];
     float sa = 0.f, sb = 0.f;
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
       const int i = threadIdx.x + j * kThreads;
       if (i < nvec) {
         e[j] = V4<T>::load(br + 4 * i);
-        wa[j] = V4<float>::load(pair.wa + 4 * i);
-        wb[j] = V4<float>::load(pair.wb + 4 * i);
+        if (kAhead) {
+          wa[j] = V4<float>::load(pair.wa + 4 * i);
+          wb[j] = V4<float>::load(pair.wb + 4 * i);
+        }
         sa += ssq4(d[j]);
         sb += ssq4(e[j]);
       }
@@ -170,16 +179,15 @@ norm_chain_vec_kernel(T* __restrict__ y, float* __restrict__ h, const T* __restr
 #pragma unroll
     for (int j = 0; j < NV; ++j)
       if (threadIdx.x + j * kThreads < nvec) {
-        d[j].x = d[j].x * fa * wa[j].x + e[j].x * fb * wb[j].x;
-        d[j].y = d[j].y * fa * wa[j].y + e[j].y * fb * wb[j].y;
-        d[j].z = d[j].z * fa * wa[j].z + e[j].z * fb * wb[j].z;
-        d[j].w = d[j].w * fa * wa[j].w + e[j].w * fb * wb[j].w;
+        const int i = 4 * (threadIdx.x + j * kThreads);
+        const float4 a = kAhead ? wa[j] : V4<float>::load(pair.wa + i), b = kAhead ? wb[j] : V4<float>::load(pair.wb + i);
+        d[j].x = d[j].x * fa * a.x + e[j].x * fb * b.x;
+        d[j].y = d[j].y * fa * a.y + e[j].y * fb * b.y;
+        d[j].z = d[j].z * fa * a.z + e[j].z * fb * b.z;
+        d[j].w = d[j].w * fa * a.w + e[j].w * fb * b.w;
       }
   }
-  if (delta) {
-    if (!kAhead) load_stage(post, pw, pb);
-    apply_stage<NV, kThreads>(post, d, pw, pb, nvec, D, red);
-  }
+  if (delta) apply_stage<NV, kThreads, kAhead>(post, d, pw, pb, nvec, D, red);
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
     const int i = threadIdx.x + j * kThreads;
@@ -195,8 +203,7 @@ norm_chain_vec_kernel(T* __restrict__ y, float* __restrict__ h, const T* __restr
     }
   }
   if (yr == nullptr) return;
-  if (!kAhead) load_stage(next, nw, nb);
-  apply_stage<NV, kThreads>(next, v, nw, nb, nvec, D, red);
+  apply_stage<NV, kThreads, kAhead>(next, v, nw, nb, nvec, D, red);
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
     const int i = threadIdx.x + j * kThreads;
@@ -282,15 +289,27 @@ template <typename T>
 int launch_chain(void* y, float* h, const void* delta, const NormPair& pair, const NormStage& post, float mult,
                  const float* add, const NormStage& next, const int* row_idx, int rows, int n_src_rows, int D, bool vec,
                  int* status, cudaStream_t stream) {
-#define CCB_CHAIN(NV, TH)                                                                                          \
-  ccb_launch(norm_chain_vec_kernel<T, NV, TH>, dim3(rows), dim3(TH), 0, stream, (T*)y, h, (const T*)delta, pair, post, \
-             mult, add, next, row_idx, n_src_rows, D, status)
+#define CCB_CHAIN(NV, TH, AH)                                                                                      \
+  if (pair.second != nullptr)                                                                                       \
+    ccb_launch_ex(AH, norm_chain_vec_kernel<T, NV, TH, AH, true>, dim3(rows), dim3(TH), 0, stream, (T*)y, h, (const T*)delta, \
+               pair, post, mult, add, next, row_idx, n_src_rows, D, status);                                          \
+  else                                                                                                              \
+    ccb_launch_ex(AH, norm_chain_vec_kernel<T, NV, TH, AH, false>, dim3(rows), dim3(TH), 0, stream, (T*)y, h, (const T*)delta, \
+               pair, post, mult, add, next, row_idx, n_src_rows, D, status)
   if (vec && D <= 8192) {
-    if (D <= 512) CCB_CHAIN(1, 128);
-    else if (D <= 1024) CCB_CHAIN(1, 256);
-    else if (D <= 2048) CCB_CHAIN(1, 512);
-    else if (D <= 4096) CCB_CHAIN(2, 512);
-    else CCB_CHAIN(4, 512);
+    if (rows <= 148) {
+      if (D <= 512) { CCB_CHAIN(1, 128, true); }
+      else if (D <= 1024) { CCB_CHAIN(1, 256, true); }
+      else if (D <= 2048) { CCB_CHAIN(1, 512, true); }
+      else if (D <= 4096) { CCB_CHAIN(2, 512, true); }
+      else { CCB_CHAIN(4, 512, false); }
+    } else {
+      if (D <= 512) { CCB_CHAIN(1, 128, false); }
+      else if (D <= 1024) { CCB_CHAIN(1, 256, false); }
+      else if (D <= 2048) { CCB_CHAIN(2, 256, false); }
+      else if (D <= 4096) { CCB_CHAIN(4, 256, false); }
+      else { CCB_CHAIN(4, 512, false); }
+    }
     return ccb_launch_status();
   }
 #undef CCB_CHAIN

@@ -987,7 +987,7 @@ def qk_rows(rows, q_out, k_cache, v_cache, conv_w, taps: int, state, q_w, k_w, e
             positions, slot_map, entry_of_token, cu_q, state_slot, n_entries: int, status=None) -> None:
     """From the rows of a q | k product [T, (nq + nkv) * hd] to the queries ``q_out`` [T, nq, hd] and the cached keys
     and values, where the values are the keys as the convolution leaves them and the norms of q and k run over the
-    whole projection (``qk_rows.cu``).  ``conv_w`` float [taps, channels] or None; ``state`` [slots, taps - 1,
+    whole projection (``qk_rows.cu``).  ``conv_w`` [taps, channels] in the compute type or None; ``state`` [slots, taps - 1,
     channels]; ``q_w`` [nq * hd] and ``k_w`` [nkv * hd] float or None; ``n_real`` the channels of a head that count in
     the norms' means.  Requests that bring several tokens have their state moved on by ``conv_state_rows``."""
     _cuda(q_out, k_cache, v_cache, conv_w, state, q_w, k_w, inv_freq, positions, slot_map, entry_of_token, cu_q, state_slot,
@@ -997,7 +997,7 @@ def qk_rows(rows, q_out, k_cache, v_cache, conv_w, taps: int, state, q_w, k_w, e
     C = (nq + nkv) * hd
     assert rows.is_cuda and rows.stride(1) == 1 and rows.shape[0] == T and rows.shape[1] >= C and hd2 == hd
     assert rows.dtype == q_out.dtype == k_cache.dtype == v_cache.dtype and v_cache.shape == k_cache.shape
-    assert conv_w is None or (conv_w.dtype == torch.float32 and conv_w.shape == (taps, C))
+    assert conv_w is None or (conv_w.dtype == rows.dtype and conv_w.shape == (taps, C))
     assert taps == 1 or (state is not None and state.dtype == rows.dtype and tuple(state.shape[1:]) == (taps - 1, C))
     assert all(w is None or (w.dtype == torch.float32 and w.numel() == n) for w, n in
                ((q_w, nq * hd), (k_w, nkv * hd), (inv_freq, hd // 2)))

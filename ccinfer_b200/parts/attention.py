@@ -291,7 +291,8 @@ class GroupedQueryAttention(Mixer):
             convs = [qk("q_conv", self.nq), qk("k_conv", self.nkv)]
             if not self.keys_as_values:
                 convs.append(laid_out(fetch(n["v_conv"]), self.nkv, self.v_dim))
-            self.conv_w = torch.cat(convs, dim=0).float().t().contiguous()
+            conv_dtype = rt.dtype if self.keys_as_values else torch.float32
+            self.conv_w = torch.cat(convs, dim=0).to(conv_dtype).t().contiguous()
         if self.sink_score is not None:
             self.sink = torch.full((self.nq,), self.sink_score, dtype=torch.float32, device=rt.device)
         if "sink" in n:
