@@ -382,11 +382,23 @@ __global__ void embed_pair_kernel(float* __restrict__ h, T* __restrict__ rows, c
     pr = pair_table + (size_t)row * D;
   }
   const T* er = table + (size_t)id * D;
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
-    float v = to_f32(er[d]) * scale;
-    if (pr) v += to_f32(pr[d]);
-    out[d] = v;
-    if (out2) out2[d] = from_f32<T>(v);
+  constexpr int kAtOnce = 8;   // loads in flight a thread
+  for (int d0 = threadIdx.x; d0 < D; d0 += kAtOnce * blockDim.x) {
+    float v[kAtOnce], p[kAtOnce];
+#pragma unroll
+    for (int k = 0; k < kAtOnce; ++k) {
+      const int d = d0 + k * blockDim.x;
+      v[k] = d < D ? to_f32(er[d]) : 0.f;
+      p[k] = d < D && pr ? to_f32(pr[d]) : 0.f;
+    }
+#pragma unroll
+    for (int k = 0; k < kAtOnce; ++k) {
+      const int d = d0 + k * blockDim.x;
+      if (d >= D) break;
+      const float x = v[k] * scale + p[k];
+      out[d] = x;
+      if (out2) out2[d] = from_f32<T>(x);
+    }
   }
 }
 
@@ -413,7 +425,7 @@ CCB_API int ccb_embed_pair(float* h, void* rows, const void* table, const void* 
   if (D <= 0 || V <= 0 || (pair_table != nullptr && (buckets <= 0 || mul_prev < 0 || mul_cur < 0)))
     return CCB_REFUSE_SIZE;
   if (pair_table != nullptr && prev_token == nullptr) return CCB_REFUSE_ARG;
-  const int threads = D >= 1024 ? 256 : 128;
+  const int threads = D >= 2048 ? 512 : (D >= 1024 ? 256 : 128);
   if (dtype == CCB_F32)
     ccb_launch(embed_pair_kernel<float>, T_, threads, 0, stream, h, (float*)rows, (const float*)table,
                (const float*)pair_table, ids, positions, entry_of_token, cu_q, state_slot, (const int*)prev_token, scale,
