@@ -339,6 +339,14 @@ CCB_API int ccb_gelu_gate_rows(void* g, int ldg, const void* table, int ldt, int
 // theirs in the step.  `rows` (optional): the same values in the storage type, for a block that reads the stream
 // itself.  embed_pair_commit then stores each request's last token of the step (a kernel of its own: the first
 // token's block of a request may run after the last one's).
+__device__ __forceinline__ float4 quad(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 quad(const __nv_bfloat16* p) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+
 template <typename T>
 __global__ void embed_pair_kernel(float* __restrict__ h, T* __restrict__ rows, const T* __restrict__ table,
                                   const T* __restrict__ pair_table, const int* __restrict__ ids,
@@ -346,7 +354,7 @@ __global__ void embed_pair_kernel(float* __restrict__ h, T* __restrict__ rows, c
                                   const int* __restrict__ cu_q, const int* __restrict__ state_slot,
                                   const int* __restrict__ prev_token, float scale, int buckets, int mul_prev,
                                   int mul_cur, int D, int V, const int* __restrict__ pending, int n_pending,
-                                  int* status) {
+                                  int vec, int* status) {
   ccb::pdl_begin();
   const int t = blockIdx.x;
   float* out = h + (size_t)t * D;
@@ -382,23 +390,25 @@ __global__ void embed_pair_kernel(float* __restrict__ h, T* __restrict__ rows, c
     pr = pair_table + (size_t)row * D;
   }
   const T* er = table + (size_t)id * D;
-  constexpr int kAtOnce = 8;   // loads in flight a thread
-  for (int d0 = threadIdx.x; d0 < D; d0 += kAtOnce * blockDim.x) {
-    float v[kAtOnce], p[kAtOnce];
-#pragma unroll
-    for (int k = 0; k < kAtOnce; ++k) {
-      const int d = d0 + k * blockDim.x;
-      v[k] = d < D ? to_f32(er[d]) : 0.f;
-      p[k] = d < D && pr ? to_f32(pr[d]) : 0.f;
+  if (vec) {   // four neighbouring elements a thread
+    for (int d = 4 * threadIdx.x; d < D; d += 4 * blockDim.x) {
+      const float4 v = quad(er + d);
+      float4 p = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (pr) p = quad(pr + d);
+      const float4 x = make_float4(v.x * scale + p.x, v.y * scale + p.y, v.z * scale + p.z, v.w * scale + p.w);
+      *reinterpret_cast<float4*>(out + d) = x;
+      if (out2) {
+        out2[d] = from_f32<T>(x.x); out2[d + 1] = from_f32<T>(x.y);
+        out2[d + 2] = from_f32<T>(x.z); out2[d + 3] = from_f32<T>(x.w);
+      }
     }
-#pragma unroll
-    for (int k = 0; k < kAtOnce; ++k) {
-      const int d = d0 + k * blockDim.x;
-      if (d >= D) break;
-      const float x = v[k] * scale + p[k];
-      out[d] = x;
-      if (out2) out2[d] = from_f32<T>(x);
-    }
+    return;
+  }
+  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+    float v = to_f32(er[d]) * scale;
+    if (pr) v += to_f32(pr[d]);
+    out[d] = v;
+    if (out2) out2[d] = from_f32<T>(v);
   }
 }
 
@@ -425,15 +435,17 @@ CCB_API int ccb_embed_pair(float* h, void* rows, const void* table, const void* 
   if (D <= 0 || V <= 0 || (pair_table != nullptr && (buckets <= 0 || mul_prev < 0 || mul_cur < 0)))
     return CCB_REFUSE_SIZE;
   if (pair_table != nullptr && prev_token == nullptr) return CCB_REFUSE_ARG;
-  const int threads = D >= 2048 ? 512 : (D >= 1024 ? 256 : 128);
+  const int vec = D % 4 == 0 && ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(table) |
+                                  reinterpret_cast<uintptr_t>(pair_table)) & 15) == 0;
+  const int threads = (vec ? D / 4 : D) >= 1024 ? (T_ < 148 ? 1024 : 256) : 128;
   if (dtype == CCB_F32)
     ccb_launch(embed_pair_kernel<float>, T_, threads, 0, stream, h, (float*)rows, (const float*)table,
                (const float*)pair_table, ids, positions, entry_of_token, cu_q, state_slot, (const int*)prev_token, scale,
-               buckets, mul_prev, mul_cur, D, V, pending, n_pending, status);
+               buckets, mul_prev, mul_cur, D, V, pending, n_pending, vec, status);
   else if (dtype == CCB_BF16)
     ccb_launch(embed_pair_kernel<__nv_bfloat16>, T_, threads, 0, stream, h, (__nv_bfloat16*)rows,
                (const __nv_bfloat16*)table, (const __nv_bfloat16*)pair_table, ids, positions, entry_of_token, cu_q,
-               state_slot, (const int*)prev_token, scale, buckets, mul_prev, mul_cur, D, V, pending, n_pending, status);
+               state_slot, (const int*)prev_token, scale, buckets, mul_prev, mul_cur, D, V, pending, n_pending, vec, status);
   else
     return CCB_REFUSE_DTYPE;
   int rc = ccb_launch_status();

@@ -15,8 +15,9 @@
 // that brings ONE token has its state moved on here (conv_state_rows does it for the others, afterwards).
 // Everything between the loads and the stores is float.
 //
-// A block takes a token, or several one after another.  A unit of work is 8 channels i .. i + 7 of a head's first half and their partners i + hd / 2:
-// a thread holds its units in registers from the convolution over the norm to the rotation.
+// A block takes a token, or several one after another.  A unit of work is 8 channels i .. i + 7 of a head's first half
+// and their partners i + hd / 2: a thread holds its units in registers from the convolution over the norm to the
+// rotation.
 #include "common.cuh"
 
 using namespace ccb;
@@ -71,10 +72,11 @@ template <typename T> __device__ __forceinline__ void unpack8(const Raw<T>& r, f
 }
 
 // TAPS > 0: that many taps, every row and weight of a unit asked for before any is used; 0: any number, in a loop (or
-// no convolution).  A block takes `per_block` tokens one after another; with one unit a thread the weights of the
-// convolution stay in registers for all of them.
-template <typename T, int NU, int TAPS>
-__global__ void __launch_bounds__(kMaxThreads)
+// no convolution).  A block takes `per_block` tokens one after another.  MANY: many tokens, so the registers of a thread
+// are kept to what lets three or four blocks share an SM (a unit's halves one after the other, the taps' weights from L1);
+// else the weights of the convolution are in registers before the kernel waits for its predecessor.
+template <typename T, int NU, int TAPS, bool MANY>
+__global__ void __launch_bounds__(kMaxThreads, MANY ? 2 : 1)
 qk_rows_kernel(const T* __restrict__ in, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
                const T* __restrict__ conv_w, T* __restrict__ state, const float* __restrict__ q_w,
                const float* __restrict__ k_w, const float* __restrict__ inv_freq, const int* __restrict__ positions,
@@ -82,7 +84,7 @@ qk_rows_kernel(const T* __restrict__ in, T* __restrict__ q_out, T* __restrict__ 
                const int* __restrict__ state_slot, const QkRows a, int rows, int per_block, int* status) {
   __shared__ float2 cs_table[2][128];
   __shared__ float red[2][64];
-  constexpr bool kHeld = NU == 1 && TAPS > 0;
+  constexpr bool kHeld = NU == 1 && TAPS > 0 && !MANY;
   const int threads = blockDim.x;
   const int half = a.hd >> 1;
   const int upu = half >> 3;                       // units per head
@@ -138,7 +140,36 @@ qk_rows_kernel(const T* __restrict__ in, T* __restrict__ q_out, T* __restrict__ 
       const int u = threadIdx.x + m * threads;
       if (u < units) {
         const int head = u / upu, c0 = head * a.hd + (u - head * upu) * 8;
-        if (TAPS > 0 && live) {
+        if (TAPS > 0 && MANY && live) {
+          constexpr int TP = TAPS > 0 ? TAPS : 1;
+#pragma unroll
+          for (int s = 0; s < 2; ++s) {
+            const int c = c0 + s * half;
+            Raw<T> raw[TP], w[TP];
+#pragma unroll
+            for (int j = 0; j < TP; ++j) {
+              const int mrow = li - (TP - 1) + j;
+              const T* src = mrow >= 0 ? in + (size_t)(r0 + mrow) * a.row_stride + c
+                                       : (st != nullptr ? st + (size_t)(TP - 1 + mrow) * C + c : nullptr);
+              raw[j] = src != nullptr ? load_raw(src) : zero_raw(T());
+              w[j] = load_raw(conv_w + (size_t)j * C + c);
+            }
+#pragma unroll
+            for (int k = 0; k < 8; ++k) x[m][s][k] = 0.f;
+#pragma unroll
+            for (int j = 0; j < TP; ++j) {
+              float uu[8], ww[8];
+              unpack8(raw[j], uu);
+              unpack8(w[j], ww);
+#pragma unroll
+              for (int k = 0; k < 8; ++k) x[m][s][k] = fmaf(ww[k], uu[k], x[m][s][k]);
+            }
+            if (moves) {
+#pragma unroll
+              for (int j = 0; j + 1 < TP; ++j) store_raw(st + (size_t)j * C + c, raw[j + 1]);
+            }
+          }
+        } else if (TAPS > 0 && live) {
           constexpr int TP = TAPS > 0 ? TAPS : 1;
           Raw<T> raw[2 * TP];
 #pragma unroll
@@ -267,17 +298,21 @@ int launch_rows(const void* in, void* q_out, void* k_cache, void* v_cache, const
                 cudaStream_t stream) {
   const int units = (a.nq + a.nkv) * (a.hd >> 4);
   const int threads = ((units + NU - 1) / NU + 31) / 32 * 32;
-  // many tokens: as many a block as two blocks on every SM leave, so that the weights are fetched once for all of them
-  const int per_block = rows <= 2 * 148 ? 1 : (rows + 2 * 148 - 1) / (2 * 148);
+  // many tokens: as many a block as three blocks on every SM leave, so that the weights are fetched once for all of them
+  const bool many = rows > 2 * 148 && NU == 1;
+  const int per_block = rows <= 2 * 148 ? 1 : (rows + 3 * 148 - 1) / (3 * 148);
   const dim3 grid((rows + per_block - 1) / per_block);
 #define CCB_QK(TP)                                                                                                    \
-  ccb_launch_ex(true, qk_rows_kernel<T, NU, TP>, grid, dim3(threads), 0, stream, (const T*)in, (T*)q_out, (T*)k_cache, \
+  if (many) CCB_QKM(TP, (NU == 1)); else CCB_QKM(TP, false)
+#define CCB_QKM(TP, MM)                                                                                               \
+  ccb_launch_ex(true, qk_rows_kernel<T, NU, TP, MM>, grid, dim3(threads), 0, stream, (const T*)in, (T*)q_out, (T*)k_cache, \
                 (T*)v_cache, (const T*)conv_w, (T*)state, q_w, k_w, inv_freq, positions, slot_map, entry_of_token, cu_q, \
                 state_slot, a, rows, per_block, status)
-  if (conv_w != nullptr && a.taps == 2) CCB_QK(2);
-  else if (conv_w != nullptr && a.taps == 3) CCB_QK(3);
-  else if (conv_w != nullptr && a.taps == 4) CCB_QK(4);
-  else CCB_QK(0);
+  if (conv_w != nullptr && a.taps == 2) { CCB_QK(2); }
+  else if (conv_w != nullptr && a.taps == 3) { CCB_QK(3); }
+  else if (conv_w != nullptr && a.taps == 4) { CCB_QK(4); }
+  else { CCB_QK(0); }
+#undef CCB_QKM
 #undef CCB_QK
   return ccb_launch_status();
 }
@@ -300,8 +335,8 @@ int pick_units(const void* in, void* q_out, void* k_cache, void* v_cache, const 
 
 }  // namespace
 
-// in [T, row_stride]: the q | k product.  conv_w (storage type) null: no convolution (taps 1).  q_w [nq * hd], k_w [nkv * hd] (float,
-// null: no norm); n_real: the channels of a head that count in the norm's mean.  hd a multiple of 16 up to 256, at
+// in [T, row_stride]: the q | k product.  conv_w (storage type) null: no convolution (taps 1).  q_w [nq * hd],
+// k_w [nkv * hd] (float, null: no norm); n_real: the channels of a head that count in the norm's mean.  hd a multiple of 16 up to 256, at
 // most 32,768 channels.
 CCB_API int ccb_qk_rows(const void* in, int row_stride, void* q_out, void* k_cache, void* v_cache, const void* conv_w,
                         int taps, void* state, const float* q_w, const float* k_w, float eps, int n_real,

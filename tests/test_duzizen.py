@@ -369,6 +369,7 @@ def test_kept_first_keys_in_every_attention_kernel(which, window, keep_first):
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("nq,nkv,hd,n_real,taps,norm,rot", [
     (4, 2, 16, 16, 3, True, True), (1, 1, 32, 20, 1, True, True), (6, 2, 64, 64, 4, True, False),
+    (2, 2, 64, 60, 2, True, True), (2, 1, 16, 16, 1, True, True),
     (32, 8, 128, 128, 4, True, True), (3, 3, 48, 44, 6, False, True), (12, 12, 256, 256, 2, True, True)])
 def test_qk_rows_kernel(dtype, nq, nkv, hd, n_real, taps, norm, rot):
     """Queries, keys and values from the product's rows: a request that goes on with several tokens, one that brings
@@ -378,7 +379,7 @@ def test_qk_rows_kernel(dtype, nq, nkv, hd, n_real, taps, norm, rot):
     C, eps, page = (nq + nkv) * hd, 1e-5, 8
     rnd = lambda *s: torch.randn(*s, generator=g)
     real = (torch.arange(C) % hd < n_real).float()
-    many = 700 if hd == 64 else 3                   # (many tokens: several a block)
+    many = 700 if hd in (16, 64) else 3             # (many tokens: several a block)
     counts, starts = [1, 5, many], [6, 9, 0]        # single-token entries first, as a step lists them
     full = [(rnd(s + n, C) * real).to(dtype) for s, n in zip(starts, counts)]
     conv = (rnd(taps, C) if taps > 1 else None)
@@ -431,7 +432,8 @@ def test_qk_rows_kernel(dtype, nq, nkv, hd, n_real, taps, norm, rot):
             sm = int(slot_map[t])
             got = (q_out[t], kc[sm // page, :, sm % page], vc[sm // page, :, sm % page])
             for x, want in zip(got, (out[0], out[1], kv.view(nkv, hd))):
-                assert (x.cpu().double() - want).abs().max() < tol * max(1.0, float(want.abs().max())), t
+                # (a float angle at position i is off by up to i * 6e-8)
+                assert (x.cpu().double() - want).abs().max() < (tol + 2e-7 * i) * max(1.0, float(want.abs().max())), t
             t += 1
     if keep:
         for f, sl in zip(full, slots):
