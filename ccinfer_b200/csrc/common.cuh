@@ -100,34 +100,31 @@ __device__ __forceinline__ float row_ssq(const float* row, int n, int lane) {
 }
 
 // The gated activation of a feed-forward, as the epilogue of its gate|up product:
-//   gelu = 0, limit <= 0:  silu(g) * u
-//   gelu = 0, limit  > 0:  g' = min(g, limit), u' = clamp(u, -limit, limit);  g' * sigmoid(alpha g') * (u' + shift)
-//   gelu = 1:              gelu(g) * u with the tanh form  0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))), written
-//                          as g * sigmoid(2 sqrt(2 / pi) (g + 0.044715 g^3))
+//   g * sigmoid(g * (alpha + cubic * g^2)) * u
+// where with limit > 0 g and u are first g' = min(g, limit), u' = clamp(u, -limit, limit) + shift.
+//   silu(g) * u:     limit 0, alpha 1, cubic 0
+//   clamped:         limit, alpha and shift of the model's choosing, cubic 0
+//   gelu(g) * u with the tanh form 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))):  since 0.5 (1 + tanh(z)) =
+//                    sigmoid(2 z), alpha = 2 sqrt(2 / pi) and cubic = 0.044715 alpha
 struct CcbGluAct {
-  float limit, alpha, shift;
-  int gelu;
+  float limit, alpha, shift, cubic;
 };
 
 __device__ __forceinline__ float glu_act(const CcbGluAct a, float g, float u) {
-  if (a.gelu) return g / (1.f + __expf(-1.5957691216057308f * g * (1.f + 0.044715f * g * g))) * u;
   if (a.limit > 0.f) {
     g = fminf(g, a.limit);
-    u = fminf(fmaxf(u, -a.limit), a.limit);
-    return g / (1.f + __expf(-a.alpha * g)) * (u + a.shift);
+    u = fminf(fmaxf(u, -a.limit), a.limit) + a.shift;
   }
-  return g / (1.f + __expf(-g)) * u;
+  return g / (1.f + __expf(-g * fmaf(a.cubic, g * g, a.alpha))) * u;
 }
 
 // The same with the accurate exponential (kernels of their own, the 32-bit path).
 __device__ __forceinline__ float glu_act_exact(const CcbGluAct a, float g, float u) {
-  if (a.gelu) return g / (1.f + expf(-1.5957691216057308f * g * (1.f + 0.044715f * g * g))) * u;
   if (a.limit > 0.f) {
     g = fminf(g, a.limit);
-    u = fminf(fmaxf(u, -a.limit), a.limit);
-    return g / (1.f + expf(-a.alpha * g)) * (u + a.shift);
+    u = fminf(fmaxf(u, -a.limit), a.limit) + a.shift;
   }
-  return g / (1.f + expf(-g)) * u;
+  return g / (1.f + expf(-g * fmaf(a.cubic, g * g, a.alpha))) * u;
 }
 
 // What an attention kernel takes beside keys and values (all optional):

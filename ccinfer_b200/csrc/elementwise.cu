@@ -183,11 +183,11 @@ __global__ void gated_act_bf16x8_kernel(uint4* __restrict__ act, const uint4* __
 }
 
 CCB_API int ccb_gated_act(void* act, const void* gate_up, int T_, int F, int block, float limit, float alpha,
-                          float up_shift, int gelu, int dtype, cudaStream_t stream) {
+                          float up_shift, float cubic, int dtype, cudaStream_t stream) {
   if (T_ <= 0) return 0;
   if (F <= 0 || block < 0 || (block > 0 && F % block != 0)) return CCB_REFUSE_SIZE;
-  if (!gelu && !(limit > 0.f)) return CCB_REFUSE_ARG;
-  const CcbGluAct a{limit, alpha, up_shift, gelu};
+  if (cubic == 0.f && !(limit > 0.f)) return CCB_REFUSE_ARG;
+  const CcbGluAct a{limit, alpha, up_shift, cubic};
   const int B = block == 0 ? F : block;
   const size_t total = (size_t)T_ * F;
   const int threads = 256;

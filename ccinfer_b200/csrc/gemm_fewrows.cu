@@ -350,12 +350,12 @@ CCB_API int ccb_gemm_fewrows_bf16(void* C, const void* A, const void* W, int M, 
   return fewrows_checked(C, A, W, M, N, K, lda, ldw, ldc, out_dtype, swiglu, CcbNormFuse{}, status, stream);
 }
 
-// The gated form with one of the other activations of ccb::glu_act in place of silu(gate) * up (limit > 0, or gelu).
+// The gated form with one of the other activations of ccb::glu_act in place of silu(gate) * up (limit > 0, or cubic != 0).
 CCB_API int ccb_gemm_fewrows_glu_bf16(void* C, const void* A, const void* W, int M, int N, int K, int lda, int ldw,
-                                      int ldc, int out_dtype, float limit, float alpha, float shift, int gelu, int* status,
+                                      int ldc, int out_dtype, float limit, float alpha, float shift, float cubic, int* status,
                                       cudaStream_t stream) {
-  if (!gelu && !(limit > 0.f)) return CCB_REFUSE_ARG;
-  t_glu_act = CcbGluAct{limit, alpha, shift, gelu};
+  if (cubic == 0.f && !(limit > 0.f)) return CCB_REFUSE_ARG;
+  t_glu_act = CcbGluAct{limit, alpha, shift, cubic};
   const int rc = fewrows_checked(C, A, W, M, N, K, lda, ldw, ldc, out_dtype, 1, CcbNormFuse{}, status, stream);
   t_glu_act = CcbGluAct{0.f, 1.f, 0.f};
   return rc;

@@ -422,11 +422,11 @@ CCB_API int ccb_gemm_tc_swiglu_bf16(void* act, const void* A, const void* W, int
   return tc_swiglu(act, A, W, M, F, K, lda, ldw, ld_act, CcbRowScale{}, status, stream);
 }
 
-// The same with one of the other activations of ccb::glu_act in place of silu(gate) * up (limit > 0, or gelu).
+// The same with one of the other activations of ccb::glu_act in place of silu(gate) * up (limit > 0, or cubic != 0).
 CCB_API int ccb_gemm_tc_glu_bf16(void* act, const void* A, const void* W, int M, int F, int K, int lda, int ldw,
-                                 int ld_act, float limit, float alpha, float shift, int gelu, int* status, cudaStream_t stream) {
-  if (!gelu && !(limit > 0.f)) return CCB_REFUSE_ARG;
-  t_glu_act = CcbGluAct{limit, alpha, shift, gelu};
+                                 int ld_act, float limit, float alpha, float shift, float cubic, int* status, cudaStream_t stream) {
+  if (cubic == 0.f && !(limit > 0.f)) return CCB_REFUSE_ARG;
+  t_glu_act = CcbGluAct{limit, alpha, shift, cubic};
   const int rc = tc_swiglu(act, A, W, M, F, K, lda, ldw, ld_act, CcbRowScale{}, status, stream);
   t_glu_act = CcbGluAct{0.f, 1.f, 0.f};
   return rc;

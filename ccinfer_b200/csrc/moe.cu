@@ -672,15 +672,15 @@ CCB_API int ccb_moe_route_sort(const float* logits, int ldl, const float* correc
 // mode 0: C (the compute type) [sorted rows, N] = relu(A[src_row] W_e^T)^2 * row_w;  mode 1: C (float) = A W_e^T
 // with A's rows the sorted rows themselves;  mode 2: W_e's N rows are gate and up rows in turn, C (the compute
 // type) [sorted rows, N / 2] = glu(gate, up) * row_w, or with w_in glu(gate * row_w, up * row_w); limit, alpha, shift,
-// gelu: which glu (CcbGluAct).  Tiles of 16 rows (what moe_sort was given).
+// cubic: which glu (CcbGluAct).  Tiles of 16 rows (what moe_sort was given).
 CCB_API int ccb_moe_grouped(const void* A, int lda, const int* src_row, const void* W, int ldw,
                             long long w_expert_stride, void* C, int ldc, const float* row_w, const int* tile_e,
                             const int* tile_r0, const int* tile_n, int max_tiles, int N, int K, int BM, int mode,
-                            float limit, float alpha, float shift, int gelu, int w_in, int dtype,
+                            float limit, float alpha, float shift, float cubic, int w_in, int dtype,
                             cudaStream_t stream) {
   if (max_tiles <= 0 || N <= 0) return 0;
   if (K <= 0 || mode < 0 || mode > 2 || (mode == 2 && (N & 1))) return CCB_REFUSE_SIZE;
-  const CcbGluAct ga{limit, alpha, shift, gelu};
+  const CcbGluAct ga{limit, alpha, shift, cubic};
   if (dtype == CCB_F32) {
     if (BM != 16) return CCB_REFUSE_SIZE;
     dim3 grid(max_tiles, (N + 127) / 128);
@@ -749,10 +749,10 @@ CCB_API int ccb_moe_combine(void* out, const float* rows, const int* pair_pos, c
 // act [rows, E F + shared] from gu [rows, 2 (E F + shared)] (gate columns, then up columns): see the kernel.
 CCB_API int ccb_moe_dense_glu_act(void* act, int lda, const void* gu, int ldg, const float* dense_w,
                                   const float* shared_gate, int sg_stride, int rows, int E, int F, int shared,
-                                  float limit, float alpha, float shift, int gelu, int w_in, int dtype,
+                                  float limit, float alpha, float shift, float cubic, int w_in, int dtype,
                                   cudaStream_t stream) {
   if (rows <= 0) return 0;
-  const CcbGluAct ga{limit, alpha, shift, gelu};
+  const CcbGluAct ga{limit, alpha, shift, cubic};
   if (E < 0 || F <= 0 || shared < 0 || lda < E * F + shared || ldg < 2 * (E * F + shared)) return CCB_REFUSE_SIZE;
   if (E > 0 && dense_w == nullptr) return CCB_REFUSE_ARG;
   const int width = E * F + shared;

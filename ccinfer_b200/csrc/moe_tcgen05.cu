@@ -237,16 +237,16 @@ CCB_API int ccb_moe_gather_rows(void* out, const void* x, const int* src_row, in
 // relu(.)^2 * row_w;  mode 1: W = the second matrices side by side [N, w_cols] (expert e at column e * F, K = F),
 // C float [rows, N];  mode 2: W = the first matrices stacked with every expert's gate and up rows in turn (F rows an
 // expert, N = F), C bfloat16 [rows, N / 2] = glu(gate, up) * row_w, or with w_in glu(gate * row_w, up * row_w); limit,
-// alpha, shift, gelu: which glu (CcbGluAct).
+// alpha, shift, cubic: which glu (CcbGluAct).
 CCB_API int ccb_moe_grouped_tc(const void* A, int lda, int rows, const void* W, int ldw, int w_rows, int w_cols,
                                void* C, int ldc, const float* row_w, const int* tile_e, const int* tile_r0,
                                const int* tile_n, int max_tiles, int N, int K, int F, int mode, float limit, float alpha,
-                               float shift, int gelu, int w_in, int* status, cudaStream_t stream) {
+                               float shift, float cubic, int w_in, int* status, cudaStream_t stream) {
   if (max_tiles <= 0 || N <= 0 || rows <= 0) return 0;
   if (K <= 0 || (K & 7) || (F & 7) || (lda & 7) || (ldw & 7) || mode < 0 || mode > 2 || (mode == 2 && (N & 1)) ||
       (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(W) & 15))
     return CCB_REFUSE_SIZE;
-  const CcbGluAct ga{limit, alpha, shift, gelu};
+  const CcbGluAct ga{limit, alpha, shift, cubic};
   CUtensorMap tmA, tmB;
   if (!ccb_tensor_map_2d(A, rows, K, lda, BK, BM, &tmA) || !ccb_tensor_map_2d(W, w_rows, w_cols, ldw, BK, 256, &tmB))
     return CCB_REFUSE_ARG;

@@ -9,6 +9,7 @@ implementation.
 from __future__ import annotations
 
 import ctypes
+import math
 import threading
 from ctypes import c_float, c_int, c_longlong, c_size_t, c_void_p
 
@@ -39,11 +40,11 @@ _SIGNATURES = {
     "ccb_gemm_tc_swiglu_bf16": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                                 c_void_p],
     "ccb_gemm_tc_glu_bf16": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-                             c_float, c_int, c_void_p, c_void_p],
+                             c_float, c_float, c_void_p, c_void_p],
     "ccb_gemm_fewrows_glu_bf16": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                  c_float, c_float, c_float, c_int, c_void_p, c_void_p],
+                                  c_float, c_float, c_float, c_float, c_void_p, c_void_p],
     "ccb_gemm_tc_pair_glu_bf16": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                  c_float, c_float, c_int, c_int, c_void_p, c_void_p],
+                                  c_float, c_float, c_float, c_int, c_void_p, c_void_p],
     "ccb_gemm_fewrows_set_stages": [c_int],
     "ccb_gemm_fewrows_bf16": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                               c_void_p, c_void_p],
@@ -66,7 +67,7 @@ _SIGNATURES = {
                                    c_void_p, c_float, c_int, c_void_p, c_void_p],
     "ccb_postnorm_residual": [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_void_p, c_float,
                               c_int, c_int, c_int, c_void_p],
-    "ccb_gated_act": [c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_int, c_void_p],
+    "ccb_gated_act": [c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_int, c_void_p],
     "ccb_delta_prepare": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p,
                           c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p],
@@ -92,7 +93,7 @@ _SIGNATURES = {
     "ccb_moe_route": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                       c_int, c_int, c_int, c_float, c_void_p],
     "ccb_moe_dense_glu_act": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                              c_float, c_float, c_float, c_int, c_int, c_int, c_void_p],
+                              c_float, c_float, c_float, c_float, c_int, c_int, c_void_p],
     "ccb_conv_rows": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                       c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p,
                       c_void_p],
@@ -109,11 +110,11 @@ _SIGNATURES = {
                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float,
                            c_void_p],
     "ccb_moe_grouped": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
-                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int,
+                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float,
                         c_int, c_int, c_void_p],
     "ccb_moe_gather_rows": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "ccb_moe_grouped_tc": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p,
-                           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int,
+                           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float,
                            c_int, c_void_p, c_void_p],
     "ccb_moe_combine": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "ccb_scaled_residual": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_void_p],
@@ -393,8 +394,11 @@ class GluAct:
     ``GluAct.clamped(limit, alpha, shift)`` min(g, limit) * sigmoid(alpha min(g, limit)) * (clamp(u, -limit, limit) +
     shift); ``GluAct.gelu_tanh()`` gelu(g) * u with the tanh form of gelu."""
 
-    def __init__(self, limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0, gelu: bool = False):
-        self.args = (float(limit), float(alpha), float(shift), 1 if gelu else 0)
+    GELU_SLOPE = 2.0 * math.sqrt(2.0 / math.pi)   # 0.5 (1 + tanh(z)) = sigmoid(2 z)
+    GELU_CUBIC = 0.044715
+
+    def __init__(self, limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0, cubic: float = 0.0):
+        self.args = (float(limit), float(alpha), float(shift), float(cubic))
 
     @classmethod
     def clamped(cls, limit: float, alpha: float, shift: float) -> "GluAct":
@@ -404,7 +408,7 @@ class GluAct:
 
     @classmethod
     def gelu_tanh(cls) -> "GluAct":
-        return cls(gelu=True)
+        return cls(alpha=cls.GELU_SLOPE, cubic=cls.GELU_CUBIC * cls.GELU_SLOPE)
 
 
 _SILU_GLU = GluAct()
