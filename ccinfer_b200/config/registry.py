@@ -61,6 +61,10 @@ def _builtin():
         from ..architectures import duzizen
         from .duzizen import DuzizenConfig
         register_architecture("Duzizen", DuzizenConfig.from_json, duzizen.build_plan)
+    if "Toripel" not in _REGISTRY:
+        from ..architectures import toripel
+        from .toripel import ToripelConfig
+        register_architecture("Toripel", ToripelConfig.from_json, toripel.build_plan)
     if "Dufizen" not in _REGISTRY:
         from ..architectures import dufizen
         from .dufizen import DufizenConfig

@@ -43,6 +43,7 @@ GROUPS = {
         "elementwise.cu",
         "norm.cu",
         "norm_chain.cu",
+        "streams.cu",
         "rope_kv.cu",
         "gemm_f32.cu",
         "gemm_cublas.cu",
@@ -67,6 +68,7 @@ GROUPS = {
         "scalar_memory.cu",
         "memory_chunks.cu",
         "delta_rule.cu",
+        "delta_head.cu",
         "linear_attention.cu",
         "ssm.cu",
     ],

@@ -272,17 +272,20 @@ __device__ __forceinline__ float lanes_sum(float v) {
 //
 // DELTA false: the plain gated recurrence  S <- diag(g_t) S + k_t v_t^T,  o_t = S^T q_t  (gated linear
 // attention): u = v, so S^T k and beta are not needed and the chain per token is the decay and one update.
-template <int R, int C, bool DELTA>
+//
+// HEAD: one decay per head and token (gg [T, H]), the same for every key channel: it is staged beside beta.
+template <int R, int C, bool DELTA, bool HEAD>
 __global__ void __launch_bounds__(kRecThreads)
 delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ vv,
                         const float* __restrict__ gg, const float* __restrict__ bb, float* __restrict__ state,
                         float* __restrict__ out, const int* __restrict__ cu_q, const int* __restrict__ state_slot,
-                        int G, int H, int dk, int dv, int tch, int g_dk) {
+                        int entry0, int G, int H, int dk, int dv, int tch) {
   ccb::pdl_begin();
+  constexpr int ROWS = HEAD ? 2 : 3;   // rows of DP floats a token is staged with: q, k (and g)
   constexpr int DP = R * kLanes;
   constexpr int COLS = kCols * C;   // columns of S per block
   extern __shared__ __align__(16) float smem[];
-  const int e = blockIdx.z, head = blockIdx.y;
+  const int e = entry0 + blockIdx.z, head = blockIdx.y;
   const int slot = state_slot[e];
   if (slot < 0) return;
   const int r0 = cu_q[e], n = cu_q[e + 1] - r0;
@@ -291,8 +294,10 @@ delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ 
   const int lane = threadIdx.x & (kLanes - 1);
   const int cl = threadIdx.x / kLanes;
   const int col0 = blockIdx.x * COLS + cl * C;   // this thread's columns: col0 .. col0 + C - 1
-  // a stage: q, k, g rows [tch][DP] each, then v [tch][COLS], then beta [tch] (padded to a multiple of 4)
-  const int stage_floats = tch * (3 * DP + COLS) + ((tch + 3) & ~3);
+  // a stage: q, k (, g) rows [tch][DP] each, then v [tch][COLS], then beta and a head's decay [tch] each (padded to a
+  // multiple of 4)
+  const int tpad = (tch + 3) & ~3;
+  const int stage_floats = tch * (ROWS * DP + COLS) + 2 * tpad;
   auto sq = [&](int s) { return smem + (size_t)s * stage_floats; };
 
   // rows past dk never change: q = k = 0, g = 1 there (the loads never touch them)
@@ -302,7 +307,7 @@ delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ 
       if (i % DP >= dk) {
         base[i] = 0.f;
         base[tch * DP + i] = 0.f;
-        base[2 * tch * DP + i] = 1.f;
+        if (!HEAD) base[2 * tch * DP + i] = 1.f;
       }
     }
   }
@@ -316,10 +321,9 @@ delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ 
       const size_t row = (size_t)(r0 + t0 + tt);
       cp_async4(base + tt * DP + r, qn + (row * G + kvh) * dk + r);
       cp_async4(base + tch * DP + tt * DP + r, kn + (row * G + kvh) * dk + r);
-      // (g_dk = 1: one decay per head and token, the same for every key channel)
-      cp_async4(base + 2 * tch * DP + tt * DP + r, gg + (row * H + head) * g_dk + (g_dk > 1 ? r : 0));
+      if (!HEAD) cp_async4(base + 2 * tch * DP + tt * DP + r, gg + (row * H + head) * dk + r);
     }
-    float* sv = base + 3 * tch * DP;
+    float* sv = base + ROWS * tch * DP;
     for (int i = threadIdx.x; i < cnt * COLS; i += kRecThreads) {
       const int tt = i / COLS, c = i - tt * COLS;
       const int gc = blockIdx.x * COLS + c;
@@ -328,6 +332,8 @@ delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ 
     float* sb = sv + tch * COLS;
     if (DELTA || bb != nullptr)
       for (int i = threadIdx.x; i < cnt; i += kRecThreads) cp_async4(sb + i, bb + (size_t)(r0 + t0 + i) * H + head);
+    if (HEAD)
+      for (int i = threadIdx.x; i < cnt; i += kRecThreads) cp_async4(sb + tpad + i, gg + (size_t)(r0 + t0 + i) * H + head);
     cp_async_commit();
   };
 
@@ -348,15 +354,16 @@ delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ 
     __syncthreads();  // chunk ch is in stage ch & 1; everyone is done with stage (ch + 1) & 1
     if (ch + 1 < chunks) fetch(ch + 1, (ch + 1) & 1);
     const float* base = sq(ch & 1);
-    const float* sv = base + 3 * tch * DP;
+    const float* sv = base + ROWS * tch * DP;
     const float* sb = sv + tch * COLS;
     const int cnt = min(tch, n - ch * tch);
 #pragma unroll 2
     for (int tt = 0; tt < cnt; ++tt) {
-      float qr[R], kr[R], gr[R];
+      float qr[R], kr[R], gr[HEAD ? 1 : R];
       Rows<R>::load(base + tt * DP, lane, qr);
       Rows<R>::load(base + tch * DP + tt * DP, lane, kr);
-      Rows<R>::load(base + 2 * tch * DP + tt * DP, lane, gr);
+      if constexpr (HEAD) gr[0] = sb[tpad + tt];
+      else Rows<R>::load(base + 2 * tch * DP + tt * DP, lane, gr);
       const float beta = (DELTA || bb != nullptr) ? sb[tt] : 1.f;   // (plain form with bb: the write is beta * v)
       constexpr int P = R < 4 ? R : 4;   // partial sums per lane
       float kqp[P];
@@ -375,7 +382,7 @@ delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ 
         for (int p = 0; p < P; ++p) dkp[p] = dqp[p] = 0.f;
 #pragma unroll
         for (int i = 0; i < R; ++i) {
-          S[c][i] *= gr[i];
+          S[c][i] *= gr[HEAD ? 0 : i];
           if (DELTA) dkp[i % P] = fmaf(S[c][i], kr[i], dkp[i % P]);
           dqp[i % P] = fmaf(S[c][i], qr[i], dqp[i % P]);
         }
@@ -541,25 +548,25 @@ CCB_API int ccb_conv_state_update(const void* proj, int ld, int oq, int ok, int 
   return ccb_launch_status();
 }
 
-template <int R, int C, bool DELTA>
+template <int R, int C, bool DELTA, bool HEAD>
 static void launch_recurrence(const float* qn, const float* kn, const float* vv, const float* gg, const float* bb,
-                              float* state, float* out, const int* cu_q, const int* state_slot, int n_entries, int G,
-                              int H, int dk, int dv, cudaStream_t stream, int g_dk) {
+                              float* state, float* out, const int* cu_q, const int* state_slot, int entry0,
+                              int n_entries, int G, int H, int dk, int dv, cudaStream_t stream) {
   constexpr int DP = R * kLanes, COLS = kCols * C;
   const int tch = DP <= 128 ? 16 : 8;
-  const size_t smem = (size_t)2 * (tch * (3 * DP + COLS) + ((tch + 3) & ~3)) * sizeof(float);
-  cudaFuncSetAttribute(delta_recurrence_kernel<R, C, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const size_t smem = (size_t)2 * (tch * ((HEAD ? 2 : 3) * DP + COLS) + 2 * ((tch + 3) & ~3)) * sizeof(float);
+  cudaFuncSetAttribute(delta_recurrence_kernel<R, C, DELTA, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                       (int)smem);
   dim3 grid((dv + COLS - 1) / COLS, H, n_entries);
-  ccb_launch(delta_recurrence_kernel<R, C, DELTA>, grid, dim3(kRecThreads), smem, stream, qn, kn, vv, gg, bb, state, out,
-             cu_q, state_slot, G, H, dk, dv, tch, g_dk);
+  ccb_launch(delta_recurrence_kernel<R, C, DELTA, HEAD>, grid, dim3(kRecThreads), smem, stream, qn, kn, vv, gg, bb,
+             state, out, cu_q, state_slot, entry0, G, H, dk, dv, tch);
 }
 
-template <bool DELTA>
+template <bool DELTA, bool HEAD>
 static int pick_recurrence(const float* qn, const float* kn, const float* vv, const float* gg, const float* bb,
                            float* state, float* out, const int* cu_q, const int* state_slot, int n_entries, int G,
-                           int H, int dk, int dv, cudaStream_t stream, bool head_decay = false) {
+                           int H, int dk, int dv, cudaStream_t stream, int entry0 = 0) {
   if (n_entries <= 0) return 0;
-  const int g_dk = head_decay ? 1 : dk;
   if (G <= 0 || H <= 0 || H % G || dk <= 0 || dk > 256 || dv <= 0) return CCB_REFUSE_SIZE;
   int R = 1;
   while (R * kLanes < dk) R *= 2;
@@ -569,7 +576,8 @@ static int pick_recurrence(const float* qn, const float* kn, const float* vv, co
   // fewer warps per SM.  Sixteen lanes a column (twice the warps, one shuffle more per sum) were no faster
   // either (1.03 ms).
 #define CCB_REC(RR) \
-  launch_recurrence<RR, 1, DELTA>(qn, kn, vv, gg, bb, state, out, cu_q, state_slot, n_entries, G, H, dk, dv, stream, g_dk)
+  launch_recurrence<RR, 1, DELTA, HEAD>(qn, kn, vv, gg, bb, state, out, cu_q, state_slot, entry0, n_entries, G, H, dk, dv, \
+                                        stream)
   switch (R) {
     case 1: CCB_REC(1); break;
     case 2: CCB_REC(2); break;
@@ -585,15 +593,25 @@ static int pick_recurrence(const float* qn, const float* kn, const float* vv, co
 CCB_API int ccb_delta_recurrence(const float* qn, const float* kn, const float* vv, const float* gg,
                                  const float* bb, float* state, float* out, const int* cu_q, const int* state_slot,
                                  int n_entries, int G, int H, int dk, int dv, cudaStream_t stream) {
-  return pick_recurrence<true>(qn, kn, vv, gg, bb, state, out, cu_q, state_slot, n_entries, G, H, dk, dv, stream);
+  return pick_recurrence<true, false>(qn, kn, vv, gg, bb, state, out, cu_q, state_slot, n_entries, G, H, dk, dv, stream);
+}
+
+// The same with one decay per head and token (gg [T, H]), for the entries entry0 .. entry0 + n_entries - 1.
+CCB_API int ccb_delta_head_recurrence(const float* qn, const float* kn, const float* vv, const float* gg,
+                                      const float* bb, float* state, float* out, const int* cu_q,
+                                      const int* state_slot, int entry0, int n_entries, int G, int H, int dk, int dv,
+                                      cudaStream_t stream) {
+  if (entry0 < 0) return CCB_REFUSE_SIZE;
+  return pick_recurrence<true, true>(qn, kn, vv, gg, bb, state, out, cu_q, state_slot, n_entries, G, H, dk, dv, stream,
+                                     entry0);
 }
 
 // The plain gated recurrence (no correction by what the state already holds): S <- diag(g) S + k v^T, o = S^T q.
 CCB_API int ccb_gated_linear_recurrence(const float* qn, const float* kn, const float* vv, const float* gg,
                                         float* state, float* out, const int* cu_q, const int* state_slot,
                                         int n_entries, int G, int H, int dk, int dv, cudaStream_t stream) {
-  return pick_recurrence<false>(qn, kn, vv, gg, nullptr, state, out, cu_q, state_slot, n_entries, G, H, dk, dv,
-                                stream);
+  return pick_recurrence<false, false>(qn, kn, vv, gg, nullptr, state, out, cu_q, state_slot, n_entries, G, H, dk, dv,
+                                       stream);
 }
 
 // The plain recurrence with ONE decay per head and token and a step size on the write (a selective state space
@@ -603,8 +621,7 @@ CCB_API int ccb_ssm_recurrence(const float* qn, const float* kn, const float* vv
                                float* state, float* out, const int* cu_q, const int* state_slot, int n_entries,
                                int G, int H, int dk, int dv, cudaStream_t stream) {
   if (a == nullptr) return CCB_REFUSE_ARG;   // (dt null: every step size is one)
-  return pick_recurrence<false>(qn, kn, vv, a, dt, state, out, cu_q, state_slot, n_entries, G, H, dk, dv, stream,
-                                true);
+  return pick_recurrence<false, true>(qn, kn, vv, a, dt, state, out, cu_q, state_slot, n_entries, G, H, dk, dv, stream);
 }
 
 template <typename T, bool SILU>

@@ -12,7 +12,8 @@
 //
 // Two kernels:
 //   latent_prepare    a block per token: c = x / rms(x) * w and kr = rot(x') into the cache row of the token;
-//                     the rotated part of every head's query into the query rows [T, H, R + r] (float)
+//                     the rotated part of every head's query into the query rows [T, H, R + r] (float); the norm of
+//                     a second latent vector that the queries are made from
 //   latent_attention  a block per (run of `tq` query tokens of a request, group of heads): 32 cached rows at
 //                     a time are staged in shared memory as floats; a warp owns one (query, head): a lane
 //                     takes a key for the scores, then a slice of the coordinates for the weighted sum
@@ -28,69 +29,102 @@ namespace {
 
 constexpr int kPrepThreads = 128;
 
-// proj [T, ld]: columns q at oq (H heads of [d | r]) and the latent row at oc ([R | r]).
-// cache [slots, R + r]; qa [T, H, R + r] float (only the last r of each head are written here).
+// proj [T, ld]: the latent row at oc ([R | r]); q [T, ldq]: the queries' rows (H heads of [d | r]), the same tensor or
+// another.  cache [slots, R + r]; qa [T, H, R + r] float (only the last r of each head are written here).
+// Each of three jobs may be left out: the cache row (slot_map null), the rotated query parts (q null), and the norm of
+// a second latent vector at on (N coordinates, times wn) into cq [T, ldc] (cq null), whose places from N on are zeroed.
+// amp: the factor on cosine and sine.
 template <typename T>
-__global__ void __launch_bounds__(kPrepThreads)
-latent_prepare_kernel(const T* __restrict__ proj, int ld, int oq, int oc, const float* __restrict__ w,
-                      const float* __restrict__ inv_freq, int rot_dims, const int* __restrict__ positions,
-                      const int* __restrict__ slot_map, T* __restrict__ cache, int num_slots, float* __restrict__ qa,
-                      int H, int d, int r, int R, float eps, int* status) {
+struct LatentRows {
+  const T* proj;
+  int ld, oc;
+  const T* q;
+  int ldq;
+  const float* w;
+  const float* inv_freq;
+  int rot_dims;
+  float amp;
+  const int* positions;
+  const int* slot_map;
+  T* cache;
+  int num_slots;
+  float* qa;
+  int H, d, r, R;
+  float eps;
+  int on, N;
+  const float* wn;
+  T* cq;
+  int ldc;
+  int* status;
+};
+
+// A block (.x) per token; .y cuts its work where tokens are few: first the cache row, then the second latent vector
+// (each if there is one), then the queries' rotated parts in pieces.  All of it in one block where gridDim.y is 1.
+template <typename T>
+__global__ void __launch_bounds__(kPrepThreads) latent_prepare_kernel(const LatentRows<T> a) {
   ccb::pdl_begin();
   __shared__ float red[32];
-  const int t = blockIdx.x;
-  const int pos = positions[t];
-  const T* row = proj + (size_t)t * ld;
-  const int half = rot_dims >> 1;
-  const int slot = slot_map ? slot_map[t] : -1;
-  const bool keep = slot >= 0;
-  // the token's blocks share the work: block 0 of the row makes the cache row, the others the queries' rotated
-  // parts (all of it in one block when the grid has one block a token)
-  const int parts = gridDim.y;
-  if (blockIdx.y == 0 && keep && slot >= num_slots) set_status(status, CCB_ST_BAD_SLOT);
-  if (blockIdx.y == 0 && keep && slot < num_slots) {
+  extern __shared__ float2 turn[];   // (cos, sin) of the token's angles, with the amplitude
+  const int t = blockIdx.x, R = a.R, r = a.r;
+  const T* row = a.proj + (size_t)t * a.ld;
+  const int half = a.rot_dims >> 1;
+  const int slot = a.slot_map ? a.slot_map[t] : -1;
+  const int n_keep = a.slot_map ? 1 : 0, n_norm = a.cq ? 1 : 0;
+  const bool all = gridDim.y == 1;
+  const bool do_keep = n_keep && (all || blockIdx.y == 0);
+  const bool do_norm = n_norm && (all || (int)blockIdx.y == n_keep);
+  const int q_parts = all ? 1 : (int)gridDim.y - n_keep - n_norm;
+  const int q_part = all ? 0 : (int)blockIdx.y - n_keep - n_norm;
+  const bool do_q = a.q != nullptr && q_part >= 0;
+  if (half > 0 && (do_keep || do_q)) {
+    const float pos = (float)a.positions[t];
+    for (int i = threadIdx.x; i < half; i += kPrepThreads) {
+      float sn, cs;
+      sincosf(pos * a.inv_freq[i], &sn, &cs);
+      turn[i] = make_float2(cs * a.amp, sn * a.amp);
+    }
+    __syncthreads();
+  }
+  auto rotated = [&](const T* x, int i) {   // coordinate i of the r coordinates at x, turned
+    if (i >= a.rot_dims) return to_f32(x[i]);
+    const int j = i < half ? i : i - half;
+    const float2 c = turn[j];
+    const float u = to_f32(x[j]), v = to_f32(x[j + half]);
+    return i < half ? u * c.x - v * c.y : v * c.x + u * c.y;
+  };
+  if (do_keep && slot >= a.num_slots && threadIdx.x == 0) set_status(a.status, CCB_ST_BAD_SLOT);
+  if (do_keep && slot >= 0 && slot < a.num_slots) {
     float ss = 0.f;
     for (int i = threadIdx.x; i < R; i += kPrepThreads) {
-      const float v = to_f32(row[oc + i]);
+      const float v = to_f32(row[a.oc + i]);
       ss += v * v;
     }
     ss = block_sum<kPrepThreads>(ss, red);
-    const float inv = 1.0f / sqrtf(ss / (float)R + eps);
-    T* dst = cache + (size_t)slot * (R + r);
-    for (int i = threadIdx.x; i < R; i += kPrepThreads) dst[i] = from_f32<T>(to_f32(row[oc + i]) * inv * w[i]);
-    const T* kr = row + oc + R;
-    for (int i = threadIdx.x; i < r; i += kPrepThreads) {
-      float v;
-      if (i < rot_dims) {
-        const int j = i < half ? i : i - half;
-        float sn, cs;
-        sincosf((float)pos * inv_freq[j], &sn, &cs);
-        const float a = to_f32(kr[j]), b = to_f32(kr[j + half]);
-        v = i < half ? a * cs - b * sn : b * cs + a * sn;
-      } else {
-        v = to_f32(kr[i]);
-      }
-      dst[R + i] = from_f32<T>(v);
-    }
+    const float inv = 1.0f / sqrtf(ss / (float)R + a.eps);
+    T* dst = a.cache + (size_t)slot * (R + r);
+    for (int i = threadIdx.x; i < R; i += kPrepThreads) dst[i] = from_f32<T>(to_f32(row[a.oc + i]) * inv * a.w[i]);
+    for (int i = threadIdx.x; i < r; i += kPrepThreads) dst[R + i] = from_f32<T>(rotated(row + a.oc + R, i));
   }
-  const int q_total = H * r;
-  const int q_per = parts > 1 ? (q_total + parts - 2) / (parts - 1) : q_total;
-  const int q_lo = (parts > 1 && blockIdx.y > 0) ? ((int)blockIdx.y - 1) * q_per : 0;
-  const int q_hi = parts > 1 ? (blockIdx.y == 0 ? 0 : min(q_total, q_lo + q_per)) : q_total;
-  for (int i = q_lo + threadIdx.x; i < q_hi; i += kPrepThreads) {
-    const int h = i / r, k = i - h * r;
-    const T* qr = row + oq + (size_t)h * (d + r) + d;
-    float v;
-    if (k < rot_dims) {
-      const int j = k < half ? k : k - half;
-      float sn, cs;
-      sincosf((float)pos * inv_freq[j], &sn, &cs);
-      const float a = to_f32(qr[j]), b = to_f32(qr[j + half]);
-      v = k < half ? a * cs - b * sn : b * cs + a * sn;
-    } else {
-      v = to_f32(qr[k]);
+  if (do_norm) {
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < a.N; i += kPrepThreads) {
+      const float v = to_f32(row[a.on + i]);
+      ss += v * v;
     }
-    qa[((size_t)t * H + h) * (R + r) + R + k] = v;
+    ss = block_sum<kPrepThreads>(ss, red);
+    const float inv = 1.0f / sqrtf(ss / (float)a.N + a.eps);
+    T* dst = a.cq + (size_t)t * a.ldc;
+    for (int i = threadIdx.x; i < a.ldc; i += kPrepThreads)
+      dst[i] = from_f32<T>(i < a.N ? to_f32(row[a.on + i]) * inv * a.wn[i] : 0.f);
+  }
+  if (do_q) {
+    const int total = a.H * r, per = (total + q_parts - 1) / q_parts;
+    const int hi = min(total, (q_part + 1) * per);
+    const T* qrow = a.q + (size_t)t * a.ldq;
+    for (int i = q_part * per + threadIdx.x; i < hi; i += kPrepThreads) {
+      const int h = i / r, k = i - h * r;
+      a.qa[((size_t)t * a.H + h) * (R + r) + R + k] = rotated(qrow + (size_t)h * (a.d + r) + a.d, k);
+    }
   }
 }
 
@@ -556,26 +590,38 @@ int pick_attention(const float* qa, const void* cache, const float* sink, const 
 
 }  // namespace
 
-CCB_API int ccb_latent_prepare(const void* proj, int ld, int oq, int oc, const float* w, const float* inv_freq,
-                               int rot_dims, const int* positions, const int* slot_map, void* cache, int num_slots,
-                               float* qa, int T, int H, int d, int r, int R, float eps, int dtype, int* status,
-                               cudaStream_t stream) {
+// What is left out: the cache row with slot_map null, the queries with q null, the second latent vector with cq null.
+CCB_API int ccb_latent_prepare(const void* proj, int ld, int oc, const void* q, int ldq, const float* w,
+                               const float* inv_freq, int rot_dims, float amp, const int* positions,
+                               const int* slot_map, void* cache, int num_slots, float* qa, int T, int H, int d, int r,
+                               int R, float eps, int on, int N, const float* wn, void* cq, int ldc, int dtype,
+                               int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H <= 0 || d < 0 || r < 0 || R <= 0 || rot_dims < 0 || rot_dims > r || (rot_dims & 1)) return CCB_REFUSE_SIZE;
-  if (rot_dims > 0 && inv_freq == nullptr) return CCB_REFUSE_ARG;
-  // few tokens: a token's work is spread over several blocks (the cache row, and the heads' rotated parts in
-  // pieces of about 512 coordinates)
-  const int parts = T <= 64 ? 1 + min(8, (H * r + 511) / 512) : 1;
+  if (cq != nullptr && (N <= 0 || ldc < N)) return CCB_REFUSE_SIZE;
+  if ((rot_dims > 0 && (inv_freq == nullptr || positions == nullptr)) || (slot_map != nullptr && (cache == nullptr || w == nullptr)) ||
+      (cq != nullptr && wn == nullptr) || (q != nullptr && qa == nullptr))
+    return CCB_REFUSE_ARG;
+  if (slot_map == nullptr && q == nullptr && cq == nullptr) return 0;
+  // few tokens: a token's work is spread over several blocks (the cache row, the second latent vector, and the heads'
+  // rotated parts in pieces of about 512 coordinates)
+  int parts = 1;
+  if (T <= 64)
+    parts = (slot_map ? 1 : 0) + (cq ? 1 : 0) + (q ? min(8, (H * r + 511) / 512) : 0);
+  if (parts < 1) parts = 1;
   const dim3 grid(T, parts);
-  if (dtype == CCB_F32)
-    ccb_launch(latent_prepare_kernel<float>, grid, dim3(kPrepThreads), 0, stream, (const float*)proj, ld, oq, oc, w,
-               inv_freq, rot_dims, positions, slot_map, (float*)cache, num_slots, qa, H, d, r, R, eps, status);
-  else if (dtype == CCB_BF16)
-    ccb_launch(latent_prepare_kernel<__nv_bfloat16>, grid, dim3(kPrepThreads), 0, stream,
-               (const __nv_bfloat16*)proj, ld, oq, oc, w, inv_freq, rot_dims, positions, slot_map,
-               (__nv_bfloat16*)cache, num_slots, qa, H, d, r, R, eps, status);
-  else
-    return CCB_REFUSE_DTYPE;
+  const size_t smem = (size_t)(rot_dims / 2) * sizeof(float2);
+  if (smem > 40 * 1024) return CCB_REFUSE_SIZE;
+#define CCB_PREP(TT)                                                                                                  \
+  do {                                                                                                                \
+    const LatentRows<TT> a{(const TT*)proj, ld, oc, (const TT*)q, ldq, w, inv_freq, rot_dims, amp, positions, slot_map, \
+                           (TT*)cache, num_slots, qa, H, d, r, R, eps, on, N, wn, (TT*)cq, ldc, status};               \
+    ccb_launch(latent_prepare_kernel<TT>, grid, dim3(kPrepThreads), smem, stream, a);                                  \
+  } while (0)
+  if (dtype == CCB_F32) CCB_PREP(float);
+  else if (dtype == CCB_BF16) CCB_PREP(__nv_bfloat16);
+  else return CCB_REFUSE_DTYPE;
+#undef CCB_PREP
   return ccb_launch_status();
 }
 

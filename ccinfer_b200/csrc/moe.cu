@@ -1,5 +1,8 @@
 // Mixture of experts: the router's choice, and the activation of the experts' first products.
 //
+// Without a router, a table names each token id's experts, all with the same weight: moe_table_route and
+// moe_table_sort (below) stand where moe_route and moe_sort would.
+//
 // Router (float throughout): s = softmax(z) over all experts, or sigmoid(z) each (RouteRule.score_fn); choice
 // scores c = s + correction; the experts form `groups` equal groups of neighbours, a group's score is its largest
 // c, or the sum of its two largest (RouteRule.group_top), only experts of the `keep` best groups can be chosen (the
@@ -137,6 +140,44 @@ moe_route_kernel(const float* __restrict__ logits, int ldl, const float* __restr
   if (t >= rows) return;
   route_token(logits, ldl, correction, idx, wts, dense_w, t, E, groups, keep, top,
               smem + (size_t)warp * (2 * E + groups), lane, rule);
+}
+
+// What a table of experts is read with: table [vocab, top], the token of each row (-1 - s: the token last sampled for
+// request slot s) and which request a row belongs to (negative: a row that pads a replayed step; it has no experts).
+struct ExpertTable {
+  const int* table;
+  const int* ids;
+  const int* entry_of_token;   // or null
+  const int* pending;
+  int top, E, vocab, n_pending;
+  float weight;
+  int* status;
+};
+
+// The expert of choice k of row t, or -1.
+__device__ __forceinline__ int table_expert(const ExpertTable& a, int t, int k) {
+  if (a.entry_of_token != nullptr && a.entry_of_token[t] < 0) return -1;
+  int id = a.ids[t];
+  if (id < 0 && a.pending != nullptr && -1 - id < a.n_pending) id = a.pending[-1 - id];
+  const int e = id >= 0 && id < a.vocab ? a.table[(size_t)id * a.top + k] : -1;
+  if (e < 0 || e >= a.E) {
+    set_status(a.status, CCB_ST_BAD_TOKEN);
+    return -1;
+  }
+  return e;
+}
+
+// dense_w [T, E]: the weight where the table names the expert, else 0.  A thread per row and expert.
+__global__ void __launch_bounds__(256)
+moe_table_route_kernel(const ExpertTable a, float* __restrict__ dense_w, int rows) {
+  ccb::pdl_begin();
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= rows * a.E) return;
+  const int t = i / a.E, e = i - t * a.E;
+  float v = 0.f;
+  for (int k = 0; k < a.top; ++k)
+    if (table_expert(a, t, k) == e) v = a.weight;
+  dense_w[i] = v;
 }
 
 template <typename T>
@@ -336,8 +377,10 @@ constexpr int kSortThreads = 1024;
 
 // idx, wts [pairs] (pairs = tokens * top).  Outputs: src_row [pairs] (token of a sorted row), row_w [pairs],
 // pair_pos [pairs] (sorted row of a pair), tile_e / tile_r0 / tile_n [max_tiles].
-// The whole block; sm: 4 E + 2 ints of shared memory.
-__device__ __forceinline__ void sort_pairs(const int* __restrict__ idx, const float* __restrict__ wts, int pairs,
+// The whole block; sm: 4 E + 2 ints of shared memory.  expert_of(p), weight_of(p): of pair p (the expert negative: the
+// pair is left out).
+template <typename ExpertOf, typename WeightOf>
+__device__ __forceinline__ void sort_pairs(ExpertOf expert_of, WeightOf weight_of, int pairs,
                                            int top, int E, int BM, int max_tiles, int* __restrict__ src_row,
                                            float* __restrict__ row_w, int* __restrict__ pair_pos,
                                            int* __restrict__ tile_e, int* __restrict__ tile_r0,
@@ -350,7 +393,7 @@ __device__ __forceinline__ void sort_pairs(const int* __restrict__ idx, const fl
   for (int e = threadIdx.x; e < E; e += kSortStride) counts[e] = 0, cursor[e] = 0;
   __syncthreads();
   for (int p = threadIdx.x; p < pairs; p += kSortStride) {
-    const int e = idx[p];
+    const int e = expert_of(p);
     if (e >= 0 && e < E) atomicAdd(&counts[e], 1);
   }
   __syncthreads();
@@ -367,12 +410,16 @@ __device__ __forceinline__ void sort_pairs(const int* __restrict__ idx, const fl
   }
   __syncthreads();
   for (int p = threadIdx.x; p < pairs; p += kSortStride) {
-    const int e = idx[p];
+    const int e = expert_of(p);
     if (e < 0 || e >= E) { pair_pos[p] = -1; continue; }
     const int pos = offs[e] + atomicAdd(&cursor[e], 1);
     src_row[pos] = p / top;
-    row_w[pos] = wts[p];
+    row_w[pos] = weight_of(p);
     pair_pos[p] = pos;
+  }
+  for (int p = offs[E] + threadIdx.x; p < pairs; p += kSortStride) {   // (places of pairs that were left out)
+    src_row[p] = 0;
+    row_w[p] = 0.f;
   }
   for (int t = threadIdx.x; t < max_tiles; t += kSortStride) {
     int n = 0, e = 0, r0 = 0;
@@ -399,7 +446,20 @@ moe_sort_kernel(const int* __restrict__ idx, const float* __restrict__ wts, int 
                 int* __restrict__ tile_e, int* __restrict__ tile_r0, int* __restrict__ tile_n) {
   ccb::pdl_begin();
   extern __shared__ int sm[];
-  sort_pairs(idx, wts, pairs, top, E, BM, max_tiles, src_row, row_w, pair_pos, tile_e, tile_r0, tile_n, sm);
+  sort_pairs([&](int p) { return idx[p]; }, [&](int p) { return wts[p]; }, pairs, top, E, BM, max_tiles, src_row, row_w,
+             pair_pos, tile_e, tile_r0, tile_n, sm);
+}
+
+// The sort with the experts read from a table as it goes: there are no idx and wts.
+__global__ void __launch_bounds__(kSortThreads)
+moe_table_sort_kernel(const ExpertTable a, int pairs, int BM, int max_tiles, int* __restrict__ src_row,
+                      float* __restrict__ row_w, int* __restrict__ pair_pos, int* __restrict__ tile_e,
+                      int* __restrict__ tile_r0, int* __restrict__ tile_n) {
+  ccb::pdl_begin();
+  extern __shared__ int sm[];
+  sort_pairs([&](int p) { const int t = p / a.top; return table_expert(a, t, p - t * a.top); },
+             [&](int) { return a.weight; }, pairs, a.top, a.E, BM, max_tiles, src_row, row_w, pair_pos, tile_e, tile_r0,
+             tile_n, sm);
 }
 
 // Steps of few tokens: the router and the sort in one block, a warp a token (up to 32 tokens).
@@ -419,7 +479,8 @@ moe_route_sort_kernel(const float* __restrict__ logits, int ldl, const float* __
                 scratch + (size_t)warp * (2 * E + groups), lane, rule);
   __threadfence_block();
   __syncthreads();   // the choices are written: the same block sorts them
-  sort_pairs(idx, wts, rows * top, top, E, BM, max_tiles, src_row, row_w, pair_pos, tile_e, tile_r0, tile_n, sm);
+  sort_pairs([&](int p) { return idx[p]; }, [&](int p) { return wts[p]; }, rows * top, top, E, BM, max_tiles, src_row, row_w,
+             pair_pos, tile_e, tile_r0, tile_n, sm);
 }
 
 __device__ __forceinline__ uint4 ld16_or_zero(const __nv_bfloat16* p, bool ok) {
@@ -647,6 +708,35 @@ CCB_API int ccb_moe_sort(const int* idx, const float* wts, int pairs, int top, i
   cudaFuncSetAttribute(moe_sort_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   ccb_launch(moe_sort_kernel, dim3(1), dim3(kSortThreads), smem, stream, idx, wts, pairs, top, E, BM, max_tiles,
              src_row, row_w, pair_pos, tile_e, tile_r0, tile_n);
+  return ccb_launch_status();
+}
+
+// Tables of experts: dense_w float [rows, E] (weight where the table names the expert), for the form that runs every
+// expert; or ccb_moe_sort with the experts read from the table.  status: a token or an expert outside its range.
+CCB_API int ccb_moe_table_route(const int* table, const int* ids, const int* entry_of_token, const int* pending,
+                                int n_pending, int vocab, int top, int E, float weight, float* dense_w, int rows,
+                                int* status, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (top <= 0 || E <= 0 || vocab <= 0 || (long long)rows * E > 0x7fffffffll) return CCB_REFUSE_SIZE;
+  const ExpertTable a{table, ids, entry_of_token, pending, top, E, vocab, n_pending, weight, status};
+  ccb_launch(moe_table_route_kernel, dim3((rows * E + 255) / 256), dim3(256), 0, stream, a, dense_w, rows);
+  return ccb_launch_status();
+}
+
+CCB_API int ccb_moe_table_sort(const int* table, const int* ids, const int* entry_of_token, const int* pending,
+                               int n_pending, int vocab, int top, int E, float weight, int rows, int BM, int max_tiles,
+                               int* src_row, float* row_w, int* pair_pos, int* tile_e, int* tile_r0, int* tile_n,
+                               int* status, cudaStream_t stream) {
+  const int pairs = rows * top;
+  if (pairs <= 0) return 0;
+  if (E <= 0 || top <= 0 || vocab <= 0 || BM <= 0 || max_tiles < min(pairs, (pairs + BM - 1) / BM + E))
+    return CCB_REFUSE_SIZE;
+  const ExpertTable a{table, ids, entry_of_token, pending, top, E, vocab, n_pending, weight, status};
+  const size_t smem = (size_t)(4 * E + 2) * sizeof(int);
+  if (smem > 96 * 1024) return CCB_REFUSE_SIZE;
+  cudaFuncSetAttribute(moe_table_sort_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  ccb_launch(moe_table_sort_kernel, dim3(1), dim3(kSortThreads), smem, stream, a, pairs, BM, max_tiles, src_row, row_w,
+             pair_pos, tile_e, tile_r0, tile_n);
   return ccb_launch_status();
 }
 

@@ -113,9 +113,15 @@ class Engine:
         self._entry_group: Dict[int, int] = {}
         self._cache: Dict[int, Dict[str, torch.Tensor]] = {}
         self._state: Dict[int, torch.Tensor] = {}
+        # what each run entry that keeps a cache must hold: its own need, and that of the entries that read it with a
+        # mask of their own
+        needs = [plan.layers[e.layer].mixer.cache_need() for e in plan.order]
+        for i, e in enumerate(plan.order):
+            if e.cache_of is not None and needs[i] is not None and needs[e.cache_of] is not None:
+                needs[e.cache_of] = needs[e.cache_of].covering(needs[i])
         for i, e in enumerate(plan.order):
             mixer = plan.layers[e.layer].mixer
-            need = mixer.cache_need()
+            need = needs[i]
             if e.cache_of is not None:
                 if need is None:
                     raise InvalidArgument(f"order[{i}] reads a cache but its mixer keeps none")

@@ -7,7 +7,7 @@ import torch
 
 from .. import kernels
 from ..errors import DeviceFault, ExtensionMissing, ScratchMoved, Unsupported
-from ..parts.base import NormedPair, UnscaledRows
+from ..parts.base import ExpertRows, NormedPair, UnscaledRows
 
 
 class ScratchPool:
@@ -74,8 +74,9 @@ class Runtime:
 
     @staticmethod
     def rows(x):
-        """x as a plain tensor (rows that a norm left short of their factor are finished, and a pair's sum is made)."""
-        return x.finish() if isinstance(x, (UnscaledRows, NormedPair)) else x
+        """x as a plain tensor (rows that a norm left short of their factor are finished, and a pair's or the experts' sum
+        is made)."""
+        return x.finish() if isinstance(x, (UnscaledRows, NormedPair, ExpertRows)) else x
 
     def _into_stream(self, out, x, w, sink) -> bool:
         """The product as the last one of a part, with few rows: added into the residual stream by its own

@@ -76,6 +76,7 @@ class StepContext:
         self.pending_tokens = None  # int32 [slots]: the token last sampled per request slot (token id -1 - s)
         self.groups: List[GroupStep] = []
         self.host = None         # host copies of the same arrays
+        self.takes_expert_rows = False   # what sums the running part's output takes parts.base.ExpertRows
         self.residual_sink = None   # parts.base.ResidualSink offered to the last product of the part that runs
 
     def take_sink(self):

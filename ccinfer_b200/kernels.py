@@ -81,8 +81,19 @@ _SIGNATURES = {
                                     c_int, c_int, c_int, c_int, c_int, c_void_p],
     "ccb_gla_prepare": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                         c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p],
-    "ccb_latent_prepare": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
-                           c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p],
+    "ccb_latent_prepare": [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p,
+                           c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
+                           c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
+    "ccb_streams_step": [c_void_p] * 6 + [c_int, c_int] + [c_void_p] * 4 + [c_float, c_void_p] + [c_int] * 5
+                        + [c_void_p, c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p],
+    "ccb_moe_table_route": [c_void_p] * 4 + [c_int] * 4 + [c_float, c_void_p, c_int, c_void_p, c_void_p],
+    "ccb_moe_table_sort": [c_void_p] * 4 + [c_int] * 4 + [c_float, c_int, c_int, c_int] + [c_void_p] * 8,
+    "ccb_delta_head_step": [c_void_p, c_int, c_void_p, c_void_p, c_int] + [c_void_p] * 5 + [c_float] + [c_void_p] * 4
+                           + [c_int] * 7 + [c_float, c_float, c_int, c_void_p],
+    "ccb_delta_head_prepare": [c_void_p, c_int, c_void_p, c_void_p, c_int] + [c_void_p] * 12 + [c_int] * 7
+                              + [c_float, c_float, c_int, c_void_p],
+    "ccb_conv_ring_write": [c_void_p, c_int, c_void_p, c_int] + [c_void_p] * 4 + [c_int] * 8 + [c_void_p],
+    "ccb_delta_head_recurrence": [c_void_p] * 9 + [c_int] * 6 + [c_void_p],
     "ccb_latent_attention": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                              c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                              c_int, c_void_p, c_void_p],
@@ -627,6 +638,76 @@ def delta_recurrence(qn, kn, vv, gg, bb, state, out, cu_q, state_slot, n_entries
                                       _p(state_slot), n_entries, G, H, dk, dv, _stream()), "delta_recurrence")
 
 
+class HeadDelta:
+    """What the kernels of the delta rule with one decay per head (``delta_head.cu``) share: the first columns of q, k, v,
+    b, a and the gate in the projections' rows, the sizes, the convolution's weights [taps, channels of q|k|v] and the
+    decay's constants."""
+
+    def __init__(self, offsets, conv_w, A_log, dt_bias, G: int, H: int, dk: int, dv: int, q_mult: float, unit_eps: float):
+        assert len(offsets) == 6 and conv_w.dtype == A_log.dtype == dt_bias.dtype == torch.float32
+        assert conv_w.shape[1] == 2 * G * dk + H * dv and A_log.numel() == dt_bias.numel() == H
+        self.offsets = (c_int * 6)(*(int(o) for o in offsets))
+        self.conv_w, self.A_log, self.dt_bias, self.taps = conv_w, A_log, dt_bias, conv_w.shape[0]
+        self.sizes, self.q_mult, self.unit_eps = (int(G), int(H), int(dk), int(dv)), float(q_mult), float(unit_eps)
+
+    def check(self, proj, ring):
+        G, H, dk, dv = self.sizes
+        _cuda(self.conv_w, self.A_log, self.dt_bias, ring)
+        assert proj.stride(1) == 1 and ring.dtype == proj.dtype
+        assert tuple(ring.shape[1:]) == (self.taps, 2 * G * dk + H * dv)
+
+
+def delta_head_step(rule: HeadDelta, proj, ring, state, w, eps: float, positions, cu_q, state_slot, y, n_entries: int) -> None:
+    """A step's first ``n_entries`` entries, one token each, through the whole mixer between its projections: y [T, H dv]
+    = o / rms(o) * w * silu(gate); the convolution's ``ring`` [slots, taps, channels] and ``state`` float [slots, H, dv, dk]
+    move on."""
+    G, H, dk, dv = rule.sizes
+    rule.check(proj, ring)
+    _cuda(state, w, positions, cu_q, state_slot)
+    assert state.dtype == torch.float32 and state.shape[1:] == (H, dv, dk) and y.stride(1) == 1 and y.dtype == proj.dtype
+    assert w.dtype == torch.float32 and w.numel() == dv and ring.shape[0] == state.shape[0]
+    _check(lib().ccb_delta_head_step(_p(proj), proj.stride(0), rule.offsets, _p(rule.conv_w), rule.taps, _p(ring), _p(state),
+                                     _p(rule.A_log), _p(rule.dt_bias), _p(w), float(eps), _p(positions), _p(cu_q),
+                                     _p(state_slot), _p(y), y.stride(0), int(n_entries), G, H, dk, dv, ring.shape[0],
+                                     rule.q_mult, rule.unit_eps, _dt(proj), _stream()), "delta_head_step")
+
+
+def delta_head_prepare(rule: HeadDelta, proj, ring, positions, entry_of_token, cu_q, state_slot, qn, kn, vv, gg, bb,
+                       row0: int, rows: int) -> None:
+    """The recurrence's inputs for the step's rows row0 .. row0 + rows - 1: unit q and k [T, G, dk], v [T, H, dv], decay
+    and beta [T, H], all float."""
+    G, H, dk, dv = rule.sizes
+    rule.check(proj, ring)
+    _cuda(positions, entry_of_token, cu_q, state_slot, qn, kn, vv, gg, bb)
+    assert proj.shape[0] >= row0 + rows and qn.shape[0] >= row0 + rows
+    _check(lib().ccb_delta_head_prepare(_p(proj), proj.stride(0), rule.offsets, _p(rule.conv_w), rule.taps, _p(ring),
+                                        _p(rule.A_log), _p(rule.dt_bias), _p(positions), _p(entry_of_token), _p(cu_q),
+                                        _p(state_slot), _p(qn), _p(kn), _p(vv), _p(gg), _p(bb), int(row0), int(rows), G, H,
+                                        dk, dv, ring.shape[0], rule.q_mult, rule.unit_eps, _dt(proj), _stream()),
+           "delta_head_prepare")
+
+
+def conv_ring_write(rule: HeadDelta, proj, ring, positions, cu_q, state_slot, entry0: int, n_entries: int) -> None:
+    """After ``delta_head_prepare``: the last rows of the portions of entries entry0 .. into the convolution's ring."""
+    G, H, dk, dv = rule.sizes
+    rule.check(proj, ring)
+    _cuda(positions, cu_q, state_slot)
+    if rule.taps > 1 and n_entries > 0:
+        _check(lib().ccb_conv_ring_write(_p(proj), proj.stride(0), rule.offsets, rule.taps, _p(ring), _p(positions),
+                                         _p(cu_q), _p(state_slot), int(entry0), int(n_entries), G, H, dk, dv,
+                                         ring.shape[0], _dt(proj), _stream()), "conv_ring_write")
+
+
+def delta_head_recurrence(qn, kn, vv, gg, bb, state, out, cu_q, state_slot, entry0: int, n_entries: int, G: int, H: int,
+                          dk: int, dv: int) -> None:
+    """``delta_recurrence`` with one decay per head and token (gg [T, H]), for the entries entry0 .. ."""
+    _cuda(qn, kn, vv, gg, bb, state, out, cu_q, state_slot)
+    assert state.dtype == torch.float32 and state.shape[1:] == (H, dv, dk) and out.dtype == torch.float32
+    _check(lib().ccb_delta_head_recurrence(_p(qn), _p(kn), _p(vv), _p(gg), _p(bb), _p(state), _p(out), _p(cu_q),
+                                           _p(state_slot), int(entry0), int(n_entries), G, H, dk, dv, _stream()),
+           "delta_head_recurrence")
+
+
 def gated_head_rmsnorm(y, o, gate, w, H: int, dv: int, eps: float, silu_gate: bool = False) -> None:
     """y[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * w * sigmoid(gate[t, h, :]); o float, gate and y storage type.
     ``silu_gate``: the factor is gate * sigmoid(gate) instead."""
@@ -663,23 +744,37 @@ def gla_prepare(proj, offsets, a, bias, qn, kn, vv, gg, H: int, dk: int, dv: int
            "gla_prepare")
 
 
-def latent_prepare(proj, oq: int, oc: int, w, inv_freq, rot_dims: int, positions, slot_map, cache, qa, H: int,
-                   d: int, r: int, R: int, eps: float, status=None) -> None:
-    """The cache rows and the rotated query parts of latent attention from the projections' rows.
+def latent_prepare(proj, oc: int, w, inv_freq, rot_dims: int, positions, slot_map, cache, H: int, d: int, r: int,
+                   R: int, eps: float, q=None, qa=None, amp: float = 1.0, low=None, status=None) -> None:
+    """The rows of latent attention from the projections' rows, three jobs of which each may be left out.
 
-    ``proj`` [T, >=]: H query heads of [d | r] from column ``oq``, the latent row [R | r] from ``oc``.  Token t's
-    cache row (``cache`` viewed as [slots, R + r], slot_map[t]; a negative slot skips it) gets
-    [x / rms(x) * w | rot(x')]; ``qa`` float [T, H, R + r] gets rot(q's last r) in the last r places of each head.
-    The rotation turns the pairs (i, i + rot_dims / 2) of the first rot_dims coordinates by pos * inv_freq[i]."""
+    ``slot_map``: token t's cache row (``cache`` viewed as [slots, R + r], slot_map[t]; a negative slot skips it) gets
+    [x / rms(x) * w | rot(x')] from proj's columns [R | r] at ``oc``.  ``q`` ([T, >=] with H query heads of [d | r]):
+    ``qa`` float [T, H, R + r] gets rot(q's last r) in the last r places of each head.  ``low`` = (on, N, weight, rows):
+    rows [T, >= N] get proj's columns on .. on + N over their root mean square, times the weight, zeros after them.
+    The rotation turns the pairs (i, i + rot_dims / 2) of the first rot_dims coordinates by pos * inv_freq[i], with
+    cosine and sine times ``amp``."""
     _cuda(w, inv_freq, positions, slot_map, cache, qa, status)
-    T = qa.shape[0]
-    assert proj.stride(1) == 1 and proj.dtype == cache.dtype and qa.dtype == torch.float32
-    assert qa.shape == (T, H, R + r) and w.dtype == torch.float32 and w.numel() == R
+    assert proj.stride(1) == 1
+    T = proj.shape[0]
+    ldq = 0
+    if q is not None:
+        assert q.stride(1) == 1 and q.dtype == proj.dtype and q.shape[0] == T
+        assert qa.dtype == torch.float32 and qa.shape == (T, H, R + r)
+        ldq = q.stride(0)
+    if slot_map is not None:
+        assert w.dtype == torch.float32 and w.numel() == R and cache.shape[-1] == R + r and cache.dtype == proj.dtype
     assert inv_freq is None or (inv_freq.dtype == torch.float32 and inv_freq.numel() >= rot_dims // 2)
-    assert cache.shape[-1] == R + r
-    _check(lib().ccb_latent_prepare(_p(proj), proj.stride(0), oq, oc, _p(w), _p(inv_freq), rot_dims, _p(positions),
-                                    _p(slot_map), _p(cache), cache.numel() // (R + r), _p(qa), T, H, d, r, R,
-                                    float(eps), _dt(proj), _p(status), _stream()), "latent_prepare")
+    on, N, wn, cq = low if low is not None else (0, 0, None, None)
+    if cq is not None:
+        _cuda(wn)
+        assert wn.dtype == torch.float32 and wn.numel() == N and cq.dtype == proj.dtype and cq.stride(1) == 1
+        assert cq.shape[0] == T and cq.shape[1] >= N
+    _check(lib().ccb_latent_prepare(_p(proj), proj.stride(0), int(oc), _p(q), ldq, _p(w), _p(inv_freq), rot_dims,
+                                    float(amp), _p(positions), _p(slot_map), _p(cache),
+                                    cache.numel() // (R + r) if cache is not None else 0, _p(qa), T, H, d, r, R, float(eps),
+                                    int(on), int(N), _p(wn), _p(cq), cq.shape[1] if cq is not None else 0, _dt(proj),
+                                    _p(status), _stream()), "latent_prepare")
 
 
 def latent_attention(qa, cache, sink, gate, out, cu_q, pos0, entry_of_token, block_table, entry0: int, n_entries: int,
@@ -810,6 +905,41 @@ def moe_dense_act(act, dense_w, E: int, F: int, shared: int) -> None:
            "moe_dense_act")
 
 
+class ExpertTable:
+    """A table [vocab, top] of int32 that names each token id's experts, all with the weight 1 / top, and the rows of a
+    step it is read for: their token ids, which request each belongs to (negative: padding, no experts), and the tokens
+    that negative ids stand for."""
+
+    def __init__(self, table, ids, entry_of_token, pending=None):
+        _cuda(table, ids, entry_of_token, pending)
+        assert table.dtype == ids.dtype == torch.int32 and table.dim() == 2 and ids.dim() == 1
+        self.table, self.ids, self.entry_of_token, self.pending = table, ids, entry_of_token, pending
+
+    def args(self, E: int):
+        vocab, top = self.table.shape
+        return (_p(self.table), _p(self.ids), _p(self.entry_of_token), _p(self.pending),
+                0 if self.pending is None else self.pending.numel(), vocab, top, int(E), 1.0 / top)
+
+
+def moe_table_route(experts: ExpertTable, dense_w, status=None) -> None:
+    """dense_w float [T, E]: the weight of every expert for every row, zero where the table does not name it."""
+    _cuda(dense_w, status)
+    T, E = dense_w.shape
+    assert dense_w.dtype == torch.float32 and experts.ids.numel() >= T
+    _check(lib().ccb_moe_table_route(*experts.args(E), _p(dense_w), T, _p(status), _stream()), "moe_table_route")
+
+
+def moe_table_sort(experts: ExpertTable, E: int, BM: int, src_row, row_w, pair_pos, tile_e, tile_r0, tile_n,
+                   status=None) -> None:
+    """``moe_sort`` for the rows of a step whose experts stand in a table."""
+    _cuda(src_row, row_w, pair_pos, tile_e, tile_r0, tile_n, status)
+    T, top, n_tiles = experts.ids.numel(), experts.table.shape[1], tile_e.numel()
+    assert src_row.numel() >= T * top and row_w.numel() >= T * top and pair_pos.numel() >= T * top
+    assert tile_r0.numel() >= n_tiles and tile_n.numel() >= n_tiles and n_tiles >= moe_max_tiles(T * top, E, BM)
+    _check(lib().ccb_moe_table_sort(*experts.args(E), T, BM, n_tiles, _p(src_row), _p(row_w), _p(pair_pos), _p(tile_e),
+                                    _p(tile_r0), _p(tile_n), _p(status), _stream()), "moe_table_sort")
+
+
 def moe_max_tiles(pairs: int, E: int, BM: int) -> int:
     """Tiles of BM rows that the sorted (token, choice) pairs of a step can need at most."""
     return min(pairs, -(-pairs // BM) + E)   # (every tile holds a pair)
@@ -937,6 +1067,51 @@ def embed_pair(h, rows, table, pair_table, ids, positions, entry_of_token, cu_q,
                                 _p(status), _stream()), "embed_pair")
     if pair_table is not None:
         counters.own += 1   # the kernel that stores each request's last token
+
+
+MAX_STREAMS = 16
+
+
+def streams_step(y, x, n_streams: int, w=None, eps: float = 0.0, weights_in=None, delta=None, pairs=None, mix=None,
+                 weights_out=None, x_out=None, table=None, ids=None, scale: float = 1.0, pending=None, row_idx=None,
+                 n_rows: int = None, status=None) -> None:
+    """A residual stream of ``n_streams`` copies between two sublayers: x_t <- sum_s mix[s, t] x_s + weights_out[t] * d,
+    then y = RMSNorm(sum_t weights_in[t] x_t; w) (``weights_in`` None: the plain sum).
+
+    ``x`` float [T, S, D], or [T, D] where all copies are equal.  d: ``delta`` [T, D] in the storage type, or
+    ``pairs`` = (rows float [pairs, D], pair_pos int32 [T * top], top), the sum of a token's rows.  ``x_out`` [T, S, D]
+    (may be x): the new copies are written there.  ``row_idx`` (int32): y holds those rows, nothing is written back.
+    ``table`` (with ``ids``): x is None, the rows table[ids[t]] * scale are written to ``x_out`` [T, D]."""
+    _cuda(y, x, w, weights_in, delta, mix, weights_out, x_out, table, ids, pending, row_idx, status)
+    S = int(n_streams)
+    if table is not None:
+        (T, D), shared = x_out.shape, True
+        assert x is None and table.shape[1] == D and ids.dtype == torch.int32 and x_out.dtype == torch.float32
+        assert y is None or y.dtype == table.dtype
+    else:
+        T, D, shared = x.shape[0], x.shape[-1], x.dim() == 2
+        assert x.dtype == torch.float32 and (shared or x.shape[1] == S)
+        assert x_out is None or (x_out.dtype == torch.float32 and x_out.shape == (T, S, D))
+    assert delta is None or pairs is None
+    assert delta is None or (delta.shape == (T, D) and (y is None or delta.dtype == y.dtype))
+    rows_p = pos_p = None
+    top = 0
+    if pairs is not None:
+        rows_p, pos_p, top = pairs
+        _cuda(rows_p, pos_p)
+        assert rows_p.dtype == torch.float32 and rows_p.shape[1] == D and pos_p.dtype == torch.int32
+        assert pos_p.numel() >= T * top
+    for v, n in ((w, D), (weights_in, S), (weights_out, S), (mix, S * S)):
+        assert v is None or (v.dtype == torch.float32 and v.numel() == n)
+    rows = T if row_idx is None else (row_idx.numel() if n_rows is None else int(n_rows))
+    assert y is None or (y.shape[0] >= rows and y.shape[1] == D)
+    ref = y if y is not None else (delta if delta is not None else table)
+    _check(lib().ccb_streams_step(_p(y), _p(x), _p(x_out), _p(delta), _p(rows_p), _p(pos_p), int(top),
+                                  rows_p.shape[0] if rows_p is not None else 0, _p(mix), _p(weights_out), _p(weights_in),
+                                  _p(w), float(eps), _p(row_idx), rows, T, S, D, 1 if shared else 0, _p(table), _p(ids),
+                                  float(scale), table.shape[0] if table is not None else 0, _p(pending),
+                                  0 if pending is None else pending.numel(), _dt(ref) if ref is not None else F32,
+                                  _p(status), _stream()), "streams_step")
 
 
 class NormSpec:

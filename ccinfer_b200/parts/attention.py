@@ -78,7 +78,8 @@ class GroupedQueryAttention(Mixer):
                  window: Optional[int] = None, own_kv: bool = True, scale: Optional[float] = None,
                  value_dim: Optional[int] = None, float_weights: bool = False, chunk: Optional[int] = None,
                  conv_taps: int = 0, value_mix: Optional[tuple] = None, keep_first: int = 0,
-                 sink_score: Optional[float] = None, keys_as_values: bool = False):
+                 sink_score: Optional[float] = None, keys_as_values: bool = False, qk_norm_weights: bool = True,
+                 tensor_core_heads: bool = False):
         """``names``: tensor names under the keys q, k, v, o and (with qk_norm_eps) q_norm, k_norm; with
         q_bias, k_bias, v_bias the projections have biases; ``sink`` [heads]; ``gate`` [heads, hidden]; with
         ``conv_taps`` > 0 q_conv, k_conv, v_conv ([channels, taps]).  ``value_mix``: ("first", key) — this
@@ -86,13 +87,15 @@ class GroupedQueryAttention(Mixer):
         lambda the scalar tensor named ``vmix``.  ``value_dim``: size of a value head where it is
         not ``head_dim``; the position encoding is then built for ``kernel_head_dim(head_dim, value_dim)``.
         ``float_weights``: the softmax weights stay float up to their product with the values (every row
-        goes to the split kernel; the tensor-core kernels round them to bfloat16 for that product)."""
+        goes to the split kernel; the tensor-core kernels round them to bfloat16 for that product).
+        ``qk_norm_weights`` False: the norms of q and k have no weights.  ``tensor_core_heads``: heads are laid out in the
+        next size that the tensor-core kernels take, where there is one (see ``kernel_head_dim``)."""
         if num_heads % num_kv_heads:
             raise Unsupported(f"{num_heads} heads are not a multiple of {num_kv_heads} kv heads")
         self.qk_dim = int(head_dim)
         self.v_dim = int(head_dim if value_dim is None else value_dim)
-        if value_dim is not None:
-            head_dim = self.kernel_head_dim(head_dim, value_dim)
+        if value_dim is not None or tensor_core_heads:
+            head_dim = self.kernel_head_dim(head_dim, self.v_dim, tensor_core_heads)
         if head_dim % 16 or head_dim > 256:
             raise Unsupported(f"head size {head_dim}: the attention kernels take multiples of 16 up to 256")
         if window is not None and window <= 0:
@@ -100,6 +103,7 @@ class GroupedQueryAttention(Mixer):
         self.hidden, self.nq, self.nkv, self.hd = int(hidden), int(num_heads), int(num_kv_heads), int(head_dim)
         self.position, self.names = position, dict(names)
         self.qk_norm_eps, self.window, self.own_kv = qk_norm_eps, window, own_kv
+        self.qk_norm_weights = bool(qk_norm_weights)
         self.has_bias = "q_bias" in self.names
         self.chunk = int(chunk) if chunk else 0
         self.taps = int(conv_taps) if conv_taps else 0
@@ -119,6 +123,8 @@ class GroupedQueryAttention(Mixer):
         if self.sink_score is not None and "sink" in self.names:
             raise Unsupported("a learned sink together with one of a constant score")
         self.keys_as_values = bool(keys_as_values)
+        if self.keys_as_values and not self.qk_norm_weights:
+            raise Unsupported("keys that are the values: norms over the whole projections have weights")
         if self.keys_as_values and (self.qk_dim != self.v_dim or not own_kv or self.has_bias or value_mix is not None
                                     or "gate" in self.names or "talk" in self.names):
             raise Unsupported("keys that are the values: equal head sizes, keys of its own, no biases, value mixing, gate "
@@ -144,9 +150,13 @@ class GroupedQueryAttention(Mixer):
         self.rt = None
 
     @staticmethod
-    def kernel_head_dim(head_dim: int, value_dim: int) -> int:
-        """The head size the kernels run with for these query/key and value sizes."""
-        return -(-max(int(head_dim), int(value_dim)) // 16) * 16
+    def kernel_head_dim(head_dim: int, value_dim: int, tensor_core_heads: bool = False) -> int:
+        """The head size the kernels run with for these query/key and value sizes: the next multiple of 16, or with
+        ``tensor_core_heads`` the next of ``kernels.DECODE_MMA_HEAD_SIZES`` if there is one."""
+        n = max(int(head_dim), int(value_dim))
+        if tensor_core_heads and n <= max(kernels.DECODE_MMA_HEAD_SIZES):
+            return min(x for x in kernels.DECODE_MMA_HEAD_SIZES if x >= n)
+        return -(-n // 16) * 16
 
     # -- what it wants ---------------------------------------------------------
     def tensor_specs(self):
@@ -161,7 +171,7 @@ class GroupedQueryAttention(Mixer):
             if self.own_kv:
                 specs += [TensorSpec(n["k_bias"], (self.nkv * self.qk_dim,), role="vector"),
                           TensorSpec(n["v_bias"], (self.nkv * self.v_dim,), role="vector")]
-        if self.qk_norm_eps is not None:
+        if self.qk_norm_eps is not None and self.qk_norm_weights:
             nq, nkv = (self.nq, self.nkv) if self.keys_as_values else (1, 1)   # heads a weight covers
             specs.append(TensorSpec(n["q_norm"], (nq * self.qk_dim,), role="vector", init="one_plus_normal"))
             if self.own_kv:
@@ -260,7 +270,8 @@ class GroupedQueryAttention(Mixer):
                                             for name, heads_of in (("q_norm", self.nq), ("k_norm", self.nkv)))
         elif self.qk_norm_eps is not None:
             def norm_w(name):
-                w = fetch(n[name]).float()
+                w = (fetch(n[name]).float() if self.qk_norm_weights
+                     else torch.ones(self.qk_dim, dtype=torch.float32, device=rt.device))
                 if self.qk_dim != hd:
                     # the kernels divide the sum of squares by hd: 1 / sqrt(ss / d + eps) =
                     # sqrt(d / hd) / sqrt(ss / hd + eps d / hd), and the added coordinates are zero

@@ -35,8 +35,10 @@ class TensorSpec:
     # "matrix": kept in the compute type (bfloat16 or float); "vector": small
     # per-channel weights, kept in float; "table": integers, kept as int32.
     role: str = "matrix"
-    # how the random-weights mode fills it: "normal" = N(0, std), "one_plus_normal" = 1 + N(0, std)
+    # how the random-weights mode fills it: "normal" = N(0, std), "one_plus_normal" = 1 + N(0, std),
+    # "eye_plus_normal" = the unit matrix + N(0, std); a table: rows of different integers below ``below``
     init: str = "normal"
+    below: int = 0
 
 
 @dataclasses.dataclass(frozen=True)
@@ -93,6 +95,17 @@ class CacheNeed:
         shape = (int(kv_heads), int(head_dim))
         return cls((CachedTensor("k", shape, token_axis=1), CachedTensor("v", shape, token_axis=1)), window, chunk,
                    int(keep_first) if window is not None or chunk is not None else 0)
+
+    def covering(self, other: "CacheNeed") -> "CacheNeed":
+        """This need with pages that live long enough for ``other``'s queries too (a layer that reads these tensors with
+        a mask of its own): the wider window, the longer run of kept first tokens; every token where one side's mask
+        is no window or the masks are of different kinds."""
+        if self.group_key == other.group_key:
+            return self
+        if self.chunk is None and other.chunk is None and self.window is not None and other.window is not None:
+            return dataclasses.replace(self, window=max(self.window, other.window),
+                                       keep_first=max(self.keep_first, other.keep_first))
+        return dataclasses.replace(self, window=None, chunk=None, keep_first=0)
 
     @property
     def group_key(self):
@@ -159,6 +172,10 @@ class Residual:
         # over some layers starts from its input plus the embedding's rows).  A block that adds them itself
         # (in the kernel of its last sum) clears this; otherwise the engine does the addition.
         self.next_add: Optional[torch.Tensor] = None
+        # A stream kept as several copies (``parts.streams``): float [T, S, D], or None while all of them are still
+        # ``h``; and the (mix, out) weights with which ``pending`` enters them.
+        self.copies: Optional[torch.Tensor] = None
+        self.connection = None
 
 
 class UnscaledRows:
@@ -193,6 +210,22 @@ class NormedPair:
 
     def finish(self):
         return self._finish(self)
+
+
+class ExpertRows:
+    """The output of a mixture of experts before it is added up: ``rows`` float [pairs, D], ``pair_pos`` the row of each
+    token's choice.  Whoever sums it into the stream adds the rows up there (``kernels.streams_step``); ``finish()``
+    returns it as a plain tensor (``Runtime.rows`` calls it)."""
+
+    def __init__(self, rows, pair_pos, top: int, finish):
+        self.rows, self.pair_pos, self.top, self._finish = rows, pair_pos, int(top), finish
+
+    @property
+    def args(self):
+        return (self.rows, self.pair_pos, self.top)
+
+    def finish(self):
+        return self._finish()
 
 
 class ResidualSink:

@@ -1,4 +1,6 @@
-"""Gated delta rule with one decay per head and key channel: a linear-attention mixer with a state.
+"""The gated delta rule: linear-attention mixers with a state.
+
+``ChannelGatedDelta`` has one decay per head and key channel, ``HeadGatedDelta`` (below) one per head.
 
 Per head, with S [key channels, value channels] starting at zero and carried from token to token:
 
@@ -143,3 +145,97 @@ class ChannelGatedDelta(Mixer):
         kernels.gated_head_rmsnorm(y, o, ag[:, self.oga:], self.norm_w, H, dv, self.eps)
         out = rt.scratch.get(self.out_key, (rt.max_tokens, self.hidden), rt.dtype)[:T]
         return rt.linear(out, y, self.w_o)
+
+
+class HeadGatedDelta(Mixer):
+    """The same rule with ONE decay per head and full-width projections:
+
+        g = exp(-exp(A_log[h]) softplus(x Wa^T + dt_bias));   y = o / rms(o) * norm_w * silu(x Wg^T), then Wo.
+
+    All projections of x are one merged matrix, q | k | v | gate | b | a.  Single tokens take one kernel between the
+    projections and Wo (``kernels.delta_head_step``); portions of prompts a preparation, the recurrence and the output norm.
+    The convolution's state is a ring of the last ``taps`` rows of q | k | v (see ``csrc/delta_head.cu``)."""
+
+    kernel_groups = ("recurrent",)
+
+    def __init__(self, hidden: int, heads: int, kv_heads: int, key_dim: int, value_dim: int, taps: int,
+                 norm_eps: float, names: dict):
+        """``names``: tensor names under the keys q, k, v, o, g, q_conv, k_conv, v_conv, a, b, A_log, dt_bias, norm."""
+        if heads % kv_heads:
+            raise Unsupported(f"{heads} heads are not a multiple of {kv_heads} q/k heads")
+        if key_dim > 256:
+            raise Unsupported(f"key size {key_dim}: the recurrence kernel holds up to 256 key channels per column")
+        if taps < 1:
+            raise Unsupported("a convolution has at least one tap")
+        self.hidden, self.H, self.G, self.dk, self.dv = int(hidden), int(heads), int(kv_heads), int(key_dim), int(value_dim)
+        self.taps, self.eps, self.names = int(taps), float(norm_eps), dict(names)
+        self.qk_width, self.v_width = self.G * self.dk, self.H * self.dv
+        # columns of the product, each start a multiple of 8 (16 bytes in bfloat16)
+        self.oq = 0
+        self.ok = _pad8(self.qk_width)
+        self.ov = self.ok + _pad8(self.qk_width)
+        self.og = self.ov + _pad8(self.v_width)
+        self.ob = self.og + _pad8(self.v_width)
+        self.oa = self.ob + _pad8(self.H)
+        self.proj_width = self.oa + _pad8(self.H)
+        self.rt = None
+
+    def tensor_specs(self):
+        n, D, C, W = self.names, self.hidden, self.qk_width, self.v_width
+        return [TensorSpec(n["q"], (C, D)), TensorSpec(n["k"], (C, D)), TensorSpec(n["v"], (W, D)),
+                TensorSpec(n["q_conv"], (C, self.taps), role="vector"),
+                TensorSpec(n["k_conv"], (C, self.taps), role="vector"),
+                TensorSpec(n["v_conv"], (W, self.taps), role="vector"),
+                TensorSpec(n["b"], (self.H, D)), TensorSpec(n["a"], (self.H, D)),
+                TensorSpec(n["A_log"], (self.H,), role="vector"), TensorSpec(n["dt_bias"], (self.H,), role="vector"),
+                TensorSpec(n["g"], (W, D)), TensorSpec(n["norm"], (self.dv,), role="vector", init="one_plus_normal"),
+                TensorSpec(n["o"], (D, W))]
+
+    def state_need(self):
+        return [StateNeed((self.H, self.dv, self.dk), torch.float32, "S"),
+                StateNeed((self.taps, 2 * self.qk_width + self.v_width), None, "conv")]
+
+    def bind(self, rt, fetch):
+        self.rt = rt
+        n = self.names
+        w = torch.zeros((self.proj_width, self.hidden), dtype=rt.dtype, device=rt.device)
+        for off, name in ((self.oq, "q"), (self.ok, "k"), (self.ov, "v"), (self.og, "g"), (self.ob, "b"), (self.oa, "a")):
+            t = fetch(n[name])
+            w[off:off + t.shape[0]] = t
+        self.w_proj = w
+        conv_w = torch.cat([fetch(n["q_conv"]), fetch(n["k_conv"]), fetch(n["v_conv"])], dim=0).float().t().contiguous()
+        self.rule = kernels.HeadDelta((self.oq, self.ok, self.ov, self.ob, self.oa, self.og), conv_w,
+                                      fetch(n["A_log"]).float().contiguous(), fetch(n["dt_bias"]).float().contiguous(),
+                                      self.G, self.H, self.dk, self.dv, self.dk ** -0.5, UNIT_EPS)
+        self.norm_w = fetch(n["norm"]).float().contiguous()
+        self.w_o = fetch(n["o"])
+
+    def forward(self, x, step, cache, state):
+        rt = self.rt
+        x = rt.rows(x)
+        T = x.shape[0]
+        G, H, dk, dv = self.G, self.H, self.dk, self.dv
+        f32 = torch.float32
+        proj = rt.scratch.get("delta_proj", (rt.max_tokens, self.proj_width), rt.dtype)[:T]
+        rt.linear(proj, x, self.w_proj)
+        S, ring = state["S"], state["conv"]
+        y = rt.scratch.get("delta_y", (rt.max_tokens, self.v_width), rt.dtype)[:T]
+        n1, many = step.n_single, step.n_entries - step.n_single
+        if n1 > 0:
+            kernels.delta_head_step(self.rule, proj, ring, S, self.norm_w, self.eps, step.positions, step.cu_q,
+                                    step.state_slot, y, n1)
+        if many > 0:
+            qn = rt.scratch.get("delta_q", (rt.max_tokens, G, dk), f32)[:T]
+            kn = rt.scratch.get("delta_k", (rt.max_tokens, G, dk), f32)[:T]
+            vv = rt.scratch.get("delta_v", (rt.max_tokens, H, dv), f32)[:T]
+            gg = rt.scratch.get("delta_decay", (rt.max_tokens, H), f32)[:T]
+            bb = rt.scratch.get("delta_beta", (rt.max_tokens, H), f32)[:T]
+            o = rt.scratch.get("delta_o", (rt.max_tokens, H, dv), f32)[:T]
+            kernels.delta_head_prepare(self.rule, proj, ring, step.positions, step.entry_of_token, step.cu_q,
+                                       step.state_slot, qn, kn, vv, gg, bb, n1, T - n1)
+            kernels.conv_ring_write(self.rule, proj, ring, step.positions, step.cu_q, step.state_slot, n1, many)
+            kernels.delta_head_recurrence(qn, kn, vv, gg, bb, S, o, step.cu_q, step.state_slot, n1, many, G, H, dk, dv)
+            kernels.gated_head_rmsnorm(y[n1:], o[n1:], proj[n1:, self.og:self.og + self.v_width], self.norm_w, H, dv,
+                                       self.eps, silu_gate=True)
+        out = rt.scratch.get(self.out_key, (rt.max_tokens, self.hidden), rt.dtype)[:T]
+        return rt.linear(out, y, self.w_o, sink=step.take_sink())

@@ -57,6 +57,12 @@ class TokenEmbedding(Part):
         rt = self.rt
         h = rt.scratch.get("residual", (rt.max_tokens, self.hidden), torch.float32)[:step.n_tokens]
         pending = getattr(step, "pending_tokens", None)
+        if self.pair is None and hasattr(first_norm, "from_table"):   # a stream of several copies, scaled or not
+            y = first_norm.from_table(h, self.table, self.scale, step.token_ids, pending)
+            if y is not None:
+                stream = Residual(h)
+                stream.ready = (first_norm, y)
+                return stream
         if self.pair is not None or self.scale != 1.0:
             rows = None
             if isinstance(first_norm, StreamRows) and rt.dtype != torch.float32:

@@ -14,21 +14,23 @@ by position * base^(-2i / rot.dims); with ``interleaved`` the pairs are (2i, 2i 
 the same thing after the rows of Wq's rotated parts and of Wdkv's are permuted alike when they are bound (a score
 does not change when q and k are permuted alike).  ``window`` None: every earlier token is seen.  Without a gate
 tensor the heads' results are taken as they are.  ``own_kv`` False: the layer has no Wdkv and reads the rows that
-another layer of the same latent size, rotated size and rotation left in its cache.
+another layer of the same latent size, rotated size and rotation left in its cache.  ``q_rank`` N: the queries go
+through a latent vector of their own, q = Wuq (c_q / rms(c_q) * w_q) with c_q = Wdq x (N coordinates).  ``ramp_scaling``:
+slow pairs turn slower and cosine and sine carry a factor, as ``position.RotaryHalf`` has it.
 
 What a token leaves in the cache is the row [c | kr] alone.  Attention runs over those rows: the unrotated part
 of a query is carried into the latent space first, (Wuk_h^T q_h) . c = q_h . (Wuk_h c), and the weighted sum of c
-comes back out through Wuv_h afterwards (two products per head, batched over the heads).  q, the latent row and
-the gate are ONE merged product of x.
+comes back out through Wuv_h afterwards (two products per head, batched over the heads).  q (or c_q), the latent row
+and the gate are ONE merged product of x.
 """
 from __future__ import annotations
 
-import numpy as np
 import torch
 
 from .. import kernels
 from ..errors import Unsupported
 from .base import CachedTensor, CacheNeed, Mixer, TensorSpec
+from .position import RotaryHalf
 
 
 def _pad8(n: int) -> int:
@@ -39,8 +41,9 @@ class LatentAttention(Mixer):
     kernel_groups = ("latent",)
     def __init__(self, hidden: int, heads: int, dim: int, rot_dim: int, value_dim: int, rank: int, window: int,
                  scale: float, rot_base: float, rot_dims: int, norm_eps: float, names: dict,
-                 interleaved: bool = False, own_kv: bool = True):
-        """``names``: tensor names under the keys q, dkv, dkv_norm, uk, uv, sink, o and optionally g (the gate)."""
+                 interleaved: bool = False, own_kv: bool = True, q_rank: int = None, ramp_scaling: dict = None):
+        """``names``: tensor names under the keys q (with ``q_rank`` dq, dq_norm, uq instead), dkv, dkv_norm, uk, uv, sink,
+        o and optionally g (the gate)."""
         if window is not None and window <= 0:
             raise Unsupported("a window of keys is > 0 (None: every earlier token)")
         if rot_dims % 2 or not (0 <= rot_dims <= rot_dim):
@@ -56,18 +59,26 @@ class LatentAttention(Mixer):
         self.interleaved, self.own_kv = bool(interleaved), bool(own_kv)
         self.names = dict(names)
         self.has_gate = "g" in self.names
-        # columns of the merged product: q | [c' | kr'] | gate logits, each start a multiple of 8
+        self.q_rank = int(q_rank) if q_rank is not None else None
+        self.ramp_scaling = dict(ramp_scaling) if ramp_scaling is not None else None
+        self.q_width = self.H * (self.d + self.r)
+        # columns of the merged product: q or c_q | [c' | kr'] | gate logits, each start a multiple of 8
         self.oq = 0
-        self.oc = _pad8(self.H * (self.d + self.r))
-        self.og = self.oc + _pad8(self.R + self.r)
-        self.in_width = self.og + _pad8(self.H)
+        self.oc = _pad8(self.q_width if self.q_rank is None else self.q_rank)
+        self.og = self.oc + (_pad8(self.R + self.r) if self.own_kv else 0)
+        self.in_width = self.og + (_pad8(self.H) if self.has_gate else 0)
         self.rt = None
 
     def tensor_specs(self):
         n, D, H = self.names, self.hidden, self.H
-        specs = [TensorSpec(n["q"], (H * (self.d + self.r), D)),
-                 TensorSpec(n["uk"], (H * self.d, self.R)), TensorSpec(n["uv"], (H * self.dv, self.R)),
-                 TensorSpec(n["sink"], (H,), role="vector"), TensorSpec(n["o"], (D, H * self.dv))]
+        if self.q_rank is None:
+            specs = [TensorSpec(n["q"], (self.q_width, D))]
+        else:
+            specs = [TensorSpec(n["dq"], (self.q_rank, D)),
+                     TensorSpec(n["dq_norm"], (self.q_rank,), role="vector", init="one_plus_normal"),
+                     TensorSpec(n["uq"], (self.q_width, self.q_rank))]
+        specs += [TensorSpec(n["uk"], (H * self.d, self.R)), TensorSpec(n["uv"], (H * self.dv, self.R)),
+                  TensorSpec(n["sink"], (H,), role="vector"), TensorSpec(n["o"], (D, H * self.dv))]
         if self.own_kv:
             specs += [TensorSpec(n["dkv"], (self.R + self.r, D)),
                       TensorSpec(n["dkv_norm"], (self.R,), role="vector", init="one_plus_normal")]
@@ -88,12 +99,20 @@ class LatentAttention(Mixer):
             half = self.rot_dims // 2
             perm = torch.tensor([2 * i for i in range(half)] + [2 * i + 1 for i in range(half)]
                                 + list(range(self.rot_dims, self.r)), device=rt.device)
-        wq = fetch(n["q"])
+        wq = fetch(n["q"] if self.q_rank is None else n["uq"])
         if perm is not None:
             wq = wq.view(H, self.d + self.r, -1).clone()
             wq[:, self.d:] = wq[:, self.d:][:, perm]
             wq = wq.view(H * (self.d + self.r), -1)
-        w[self.oq:self.oq + wq.shape[0]] = wq
+        if self.q_rank is None:
+            w[self.oq:self.oq + wq.shape[0]] = wq
+        else:
+            t = fetch(n["dq"])
+            w[self.oq:self.oq + t.shape[0]] = t
+            self.cq_norm_w = fetch(n["dq_norm"]).float().contiguous()
+            # (rows of c_q are padded with zeros to a multiple of 8, and so are this matrix's columns)
+            self.w_uq = torch.zeros((_pad8(self.q_width), _pad8(self.q_rank)), dtype=rt.dtype, device=rt.device)
+            self.w_uq[:wq.shape[0], :self.q_rank] = wq
         if self.own_kv:
             wc = fetch(n["dkv"])
             if perm is not None:
@@ -111,11 +130,14 @@ class LatentAttention(Mixer):
         self.w_uk_t = fetch(n["uk"]).view(H, self.d, self.R).transpose(1, 2).contiguous()
         self.w_uv = fetch(n["uv"]).view(H, self.dv, self.R).contiguous()
         self.w_o = fetch(n["o"])
-        self.inv_freq = None
+        self.inv_freq, self.amp = None, 1.0
         if self.rot_dims:
-            i = np.arange(self.rot_dims // 2, dtype=np.float64)
-            f = np.power(np.float64(self.rot_base), -2.0 * i / self.rot_dims).astype(np.float32)
-            self.inv_freq = torch.from_numpy(f).to(rt.device)
+            rot = RotaryHalf(self.rot_dims, self.rot_base, ramp_scaling=self.ramp_scaling,
+                             linear_scaling=1.0 if self.ramp_scaling is None else None)   # (1: evaluated in float64)
+            rot.bind(rt, fetch)
+            self.inv_freq = rot.rotary_table()
+            amp = rot.amplitude()
+            self.amp = 1.0 if amp is None else float(amp[0])
 
     def forward(self, x, step, cache, state):
         rt = self.rt
@@ -127,10 +149,21 @@ class LatentAttention(Mixer):
         rt.linear(proj, x, self.w_in)
         qa = rt.scratch.get("latent_q", (rt.max_tokens, H, R + r), torch.float32)[:T]
         rows = cache.tensors["latent"]
-        kernels.latent_prepare(proj, self.oq, self.oc, self.norm_w, self.inv_freq, self.rot_dims, step.positions,
-                               g.slot_map if cache.own else None, rows, qa, H, d, r, R, self.eps, status=rt.status)
+        prepare = (self.oc, self.norm_w, self.inv_freq, self.rot_dims, step.positions, g.slot_map if cache.own else None,
+                   rows, H, d, r, R, self.eps)
+        if self.q_rank is None:
+            q = proj[:, self.oq:self.oq + self.q_width]
+            kernels.latent_prepare(proj, *prepare, q=q, qa=qa, amp=self.amp, status=rt.status)
+        else:
+            cq = rt.scratch.get("latent_cq", (rt.max_tokens, self.w_uq.shape[1]), rt.dtype)[:T]
+            kernels.latent_prepare(proj, *prepare, amp=self.amp, low=(self.oq, self.q_rank, self.cq_norm_w, cq),
+                                   status=rt.status)
+            q = rt.scratch.get("latent_uq", (rt.max_tokens, self.w_uq.shape[0]), rt.dtype)[:T]
+            rt.linear(q, cq, self.w_uq)
+            kernels.latent_prepare(q, *prepare[:5], None, None, *prepare[7:], q=q, qa=qa, amp=self.amp, status=rt.status)
+            q = q[:, :self.q_width]
         if d > 0:
-            qu = proj[:, self.oq:self.oq + H * (d + r)].view(T, H, d + r)[:, :, :d]
+            qu = q.view(T, H, d + r)[:, :, :d]
             rt.linear_batched(qa[:, :, :R].permute(1, 0, 2), qu.permute(1, 0, 2), self.w_uk_t)
         else:
             qa[:, :, :R].zero_()

@@ -14,6 +14,10 @@ says how logits become scores and weights (sigmoid scores, a group's score as th
 scores renormalised, a last factor); ``names["shared_gate"]``: the shared expert's result is multiplied by
 sigmoid(w_sg . x), one number per token (the row rides along as one more row of the router's matrix).
 
+``table_vocab`` V (instead of a router): a table ``names["table"]`` [V, top] names each token id's experts, all different,
+each with the weight 1 / top.  In a block that says so (``step.takes_expert_rows``) the sparse form leaves its result as
+``ExpertRows``: what sums it into the stream adds a token's rows up.
+
 Two forms, chosen by size (``sparse=`` forces one):
 
 * dense, for experts so small that launches cost more than their arithmetic: every expert on every token as ONE
@@ -34,7 +38,7 @@ import torch
 
 from .. import kernels
 from ..errors import Unsupported
-from .base import FeedForward, TensorSpec
+from .base import ExpertRows, FeedForward, TensorSpec
 
 
 class MixtureOfExperts(FeedForward):
@@ -49,8 +53,8 @@ class MixtureOfExperts(FeedForward):
 
     def __init__(self, hidden: int, experts: int, top: int, expert_ff: int, names: dict, groups: int = 1,
                  keep: int = 1, shared_ff: int = 0, activation="relu2", sparse=None, rule=None,
-                 weight_on_input: bool = False):
-        """``names``: "router", "correction" (optional), "up" and "down" (and "gate" with "swiglu") with ``{e}`` for
+                 weight_on_input: bool = False, table_vocab: int = None):
+        """``names``: "router" (or with ``table_vocab`` "table"), "correction" (optional), "up" and "down" (and "gate" with "swiglu") with ``{e}`` for
         the expert's number, "shared_up" / "shared_down" (/ "shared_gate_proj") with ``shared_ff`` > 0,
         "shared_gate" (optional)."""
         custom = isinstance(activation, kernels.GluAct)
@@ -64,6 +68,10 @@ class MixtureOfExperts(FeedForward):
         if custom and shared_ff and names.get("shared_gate"):
             raise Unsupported("a gate on the shared expert together with an activation of its own")
         self.rule = rule
+        self.table_vocab = int(table_vocab) if table_vocab is not None else None
+        if self.table_vocab is not None and (rule is not None or groups != 1 or names.get("router") or names.get("correction")
+                                             or names.get("shared_gate")):
+            raise Unsupported("experts named by a table come without a router, its rule, groups or a shared gate")
         if experts % groups or not (0 < keep <= groups) or not (0 < top <= (experts // groups) * keep):
             raise Unsupported(f"{experts} experts in {groups} groups of which {keep} are kept cannot give {top}")
         self.hidden, self.E, self.top, self.F = int(hidden), int(experts), int(top), int(expert_ff)
@@ -75,7 +83,10 @@ class MixtureOfExperts(FeedForward):
 
     def tensor_specs(self):
         n, D = self.names, self.hidden
-        specs = [TensorSpec(n["router"], (self.E, D))]
+        if self.table_vocab is not None:
+            specs = [TensorSpec(n["table"], (self.table_vocab, self.top), role="table", below=self.E)]
+        else:
+            specs = [TensorSpec(n["router"], (self.E, D))]
         if n.get("correction"):
             specs.append(TensorSpec(n["correction"], (self.E,), role="vector"))
         for e in range(self.E):
@@ -93,7 +104,8 @@ class MixtureOfExperts(FeedForward):
     def bind(self, rt, fetch):
         self.rt = rt
         n = self.names
-        self.w_router = fetch(n["router"])
+        self.table = fetch(n["table"]).contiguous() if self.table_vocab is not None else None
+        self.w_router = fetch(n["router"]) if self.table is None else None
         self.has_shared_gate = bool(self.SF and n.get("shared_gate"))
         if self.has_shared_gate:   # its logit is column E of the router's product
             self.w_router = torch.cat([self.w_router, fetch(n["shared_gate"]).view(1, -1)], dim=0).contiguous()
@@ -151,10 +163,24 @@ class MixtureOfExperts(FeedForward):
         rt = self.rt
         return rt.scratch.get("moe_logits", (rt.max_tokens, self.w_router.shape[0]), torch.float32)[:T, self.E]
 
-    def route(self, x, T, sort_into=None):
+    def _named_experts(self, T, step, sort_into):
+        """What ``route`` does, with the experts from the table."""
+        rt = self.rt
+        experts = kernels.ExpertTable(self.table, step.token_ids[:T], step.entry_of_token[:T],
+                                      getattr(step, "pending_tokens", None))
+        if sort_into is not None:
+            kernels.moe_table_sort(experts, self.E, *sort_into, status=rt.status)
+            return None, None, None
+        dense = rt.scratch.get("moe_dense", (rt.max_tokens, self.E), torch.float32)[:T]
+        kernels.moe_table_route(experts, dense, status=rt.status)
+        return None, None, dense
+
+    def route(self, x, T, sort_into=None, step=None):
         """idx int32 [T, top], wts float [T, top], dense float [T, E] for the rows of x.  ``sort_into`` (BM and the
         arrays of ``kernels.moe_sort``): the pairs are sorted by expert as well, in the same kernel where the step
         has few tokens (then there is no dense row)."""
+        if self.table is not None:
+            return self._named_experts(T, step, sort_into)
         rt = self.rt
         logits = rt.scratch.get("moe_logits", (rt.max_tokens, self.w_router.shape[0]), torch.float32)[:T]
         rt.linear(logits, x, self.w_router)
@@ -170,7 +196,7 @@ class MixtureOfExperts(FeedForward):
             kernels.moe_sort(idx, wts, self.E, *sort_into)
         return idx, wts, dense
 
-    def _forward_sparse(self, x, T):
+    def _forward_sparse(self, x, T, step):
         rt = self.rt
         E, F, D, top = self.E, self.F, self.hidden, self.top
         i32, f32 = torch.int32, torch.float32
@@ -187,7 +213,7 @@ class MixtureOfExperts(FeedForward):
         row_w = rt.scratch.get(f"moe_row_w:{top}", (max_pairs,), f32)
         pair_pos = rt.scratch.get(f"moe_pair_pos:{top}", (max_pairs,), i32)
         tiles = [rt.scratch.get(f"moe_tile{k}:{top}:{E}", (cap,), i32)[:n_tiles] for k in range(3)]
-        idx, wts, _ = self.route(x, T, sort_into=(BM, src_row, row_w, pair_pos, *tiles))
+        idx, wts, _ = self.route(x, T, sort_into=(BM, src_row, row_w, pair_pos, *tiles), step=step)
         act = rt.scratch.get(f"moe_act_rows:{top}:{F}", (max_pairs, F), rt.dtype)[:pairs]
         rows = rt.scratch.get(f"moe_out_rows:{top}", (max_pairs, D), f32)[:pairs]
         # the first product's rows an expert and its mode: with gates, gate and up rows in turn and the gated
@@ -217,17 +243,22 @@ class MixtureOfExperts(FeedForward):
             kernels.moe_dense_act(sa, wts, 0, 1, self.SF)
             shared = rt.scratch.get("moe_shared_out", (rt.max_tokens, D), rt.dtype)[:T]
             rt.linear(shared, sa, self.w_shared_down)
-        out = rt.scratch.get("ffn_out", (rt.max_tokens, D), rt.dtype)[:T]
-        kernels.moe_combine(out, rows, pair_pos, shared, top)
-        return out
+        def add_up():
+            out = rt.scratch.get("ffn_out", (rt.max_tokens, D), rt.dtype)[:T]
+            kernels.moe_combine(out, rows, pair_pos, shared, top)
+            return out
+
+        if shared is None and getattr(step, "takes_expert_rows", False):
+            return ExpertRows(rows, pair_pos, top, add_up)
+        return add_up()
 
     def forward(self, x, step):
         rt = self.rt
         x = rt.rows(x)
         T = x.shape[0]
         if self.use_sparse:
-            return self._forward_sparse(x, T)
-        _, _, dense = self.route(x, T)
+            return self._forward_sparse(x, T, step)
+        _, _, dense = self.route(x, T, step=step)
         act = rt.scratch.get("moe_act", (rt.max_tokens, self.width), rt.dtype)[:T]
         if self.glu:
             gu = rt.scratch.get("moe_gate_up", (rt.max_tokens, 2 * self.width), rt.dtype)[:T]

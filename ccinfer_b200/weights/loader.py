@@ -30,7 +30,7 @@ import torch
 
 from ..errors import ModelLoadFailed
 from ..parts.base import TensorSpec
-from .random_init import normal_tensor
+from .random_init import distinct_table, normal_tensor
 from .safetensors_io import SafetensorsFile, write_safetensors
 
 WEIGHTS_FILE = "model.safetensors"
@@ -166,14 +166,20 @@ def open_weights(model_dir: str, specs: List[TensorSpec], device, compute_dtype,
 # random weights
 # ---------------------------------------------------------------------------------------------
 def random_tensor(spec: TensorSpec, seed: int, std: float, device="cpu", dtype=torch.float32) -> torch.Tensor:
-    """One tensor of the random model: N(0, std), or 1 + N(0, std) for norm weights, in ``dtype``.
+    """One tensor of the random model: N(0, std), or 1 + N(0, std) for norm weights, in ``dtype``; for an integer table
+    rows of different numbers (int32).
 
     The values are those of the counter-based stream of (seed, tensor name) (see ``random_init``): they do
     not change with the order or the number of the other tensors, nor with where they are drawn; bfloat16
     is the float value rounded once.
     """
     if spec.role == "table":
-        raise ModelLoadFailed(f"no random rule for the integer table '{spec.name}'")
+        if spec.below < spec.shape[-1]:
+            raise ModelLoadFailed(f"no random rule for the integer table '{spec.name}'")
+        return distinct_table(spec.shape, seed, spec.name, spec.below).to(device)
+    if spec.init == "eye_plus_normal":
+        t = normal_tensor(spec.shape, seed, spec.name, std, False, torch.float32, device)
+        return (t + torch.eye(*spec.shape, dtype=torch.float32, device=device)).to(dtype)
     return normal_tensor(spec.shape, seed, spec.name, std, spec.init == "one_plus_normal", dtype, device)
 
 
@@ -191,7 +197,8 @@ def write_random_model(model_dir: str, config, seed: int, std: float = 0.02, sto
     cj["torch_dtype"] = store_dtype
     plan = arch.build_plan(config)
     os.makedirs(model_dir, exist_ok=True)
-    tensors = {s.name: random_tensor(s, seed, std).to(tdt) for s in plan.tensor_specs()}
+    tensors = {s.name: random_tensor(s, seed, std) for s in plan.tensor_specs()}
+    tensors = {n: t.to(tdt) if t.is_floating_point() else t for n, t in tensors.items()}
     write_safetensors(os.path.join(model_dir, WEIGHTS_FILE), tensors,
                       metadata={"format": "pt", "weights_seed": seed, "weights_std": std})
     with open(os.path.join(model_dir, "config.json"), "w") as f:

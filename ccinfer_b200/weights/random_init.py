@@ -120,3 +120,20 @@ def normal_tensor(shape, seed: int, name: str, std: float, add_one: bool, dtype:
         return out
     host = torch.from_numpy(normal_host(numel, seed, name, std, add_one)).view(tuple(shape))
     return host.to(dtype)
+
+
+def distinct_table(shape, seed: int, name: str, below: int) -> torch.Tensor:
+    """int32 [rows, n]: n different integers of 0 .. below - 1 in each row, from the counter stream of (seed, name): row i
+    is a shuffle's first n picks, pick j drawn from the below - j numbers left."""
+    rows, n = int(shape[0]), int(shape[1])
+    key = tensor_key(name)
+    with np.errstate(over="ignore"):
+        words = np.concatenate([np.stack(_philox(np.arange(rows, dtype=np.uint64) * np.uint64(-(-n // 4)) + np.uint64(b),
+                                                 key, seed), axis=1) for b in range(-(-n // 4))], axis=1)
+    out = np.empty((rows, n), dtype=np.int64)
+    for j in range(n):
+        pick = (words[:, j] % np.uint64(below - j)).astype(np.int64)
+        for prev in np.sort(out[:, :j], axis=1).T:      # the pick-th number not taken yet
+            pick += pick >= prev
+        out[:, j] = pick
+    return torch.from_numpy(out.astype(np.int32))
