@@ -35,10 +35,10 @@ runs one of the two other workloads of the reference's benchmark record through 
 continuous batch at the Qwen3-14B shape; four 16,384-token prompts at the Qwen3-32B shape) and prints a
 line of its own: output tokens a second, the distribution of the step calls, the pages' high water.
 
-    python bench.py --design tugelorn|dufizen|burolorn|gevovik|duzizen [--design-sizes mid,8b] [--layers L] [--design-profile]
+    python bench.py --design tugelorn|dufizen|burolorn|gevovik|duzizen|toripel [--design-sizes mid,8b] [--layers L] [--design-profile]
 
 measures another design of the package beside its closest model (Tugelorn beside Qwen3, Dufizen beside
-Tugelorn, Burolorn beside Qwen3, Gevovik beside Tugelorn, Duzizen beside Dufizen) at equal layer sizes (same width, heads, head size,
+Tugelorn, Burolorn beside Qwen3, Gevovik beside Tugelorn, Duzizen and Toripel beside Dufizen) at equal layer sizes (same width, heads, head size,
 intermediate size, vocabulary and number of layers; random weights): one prompt of 2,048 and of 8,192 tokens
 in steps of 2,048 (tokens a second) and decode steps of 1 and 8 requests after 2,048-token prompts, replayed
 from CUDA graphs (tokens a second), one JSON line per size.  With --design-profile it only runs a prompt and a
@@ -396,6 +396,34 @@ def duzizen_config(size: str, layers: int):
     return DuzizenConfig.from_json(j)
 
 
+def toripel_config(size: str, layers: int):
+    """Layers in turn: latent attention over a window of 1,024 (queries through a latent of 3/8 of the width, latent
+    size 512, 64 rotated coordinates with stretched slow pairs, a sink), every second one of which reads the rows of the
+    first; a delta rule with one decay per head (H heads, four taps); attention over a window of 1,024 without positions
+    (biases, unit heads); each with a mixture of 32 gated experts of F / 4 of which a table names 4 for every token id
+    (F intermediate channels per token); a stream of four copies."""
+    from ccinfer_b200.config.toripel import ToripelConfig
+    D, H, G, hd, F, V = DESIGN_SIZES[size]
+    latent = {"heads": H, "dim": hd - 64, "rot_dim": 64, "vdim": hd, "kv_rank": 512, "q_rank": D * 3 // 8,
+              "scale": hd ** -0.5, "mask": {"size": 1024},
+              "rot": {"dims": 64, "base": 1000000.0,
+                      "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    delta = {"heads": H, "kv_heads": H, "dim": hd, "vdim": hd, "conv": 4}
+    attention = {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": 1024}}
+    mlp = {"kind": "moe", "expert": {"ff": F // 4}, "router": {"experts": 32, "top": 4}}
+    out = []
+    for i in range(layers):
+        if i % 3 == 0:
+            mixer = dict(latent, kv_from=0) if (i // 3) % 2 == 1 else latent
+            out.append({"type": "latent_attention", "mixer": mixer, "mlp": mlp})
+        elif i % 3 == 1:
+            out.append({"type": "delta", "mixer": delta, "mlp": mlp})
+        else:
+            out.append({"type": "attention", "mixer": attention, "mlp": mlp})
+    return ToripelConfig.from_json({"architecture": "Toripel", "vocab": V, "width": D, "streams": 4,
+                                    "norm": {"eps": 1e-5}, "embedding": {"scale": D ** 0.5}, "layers": out})
+
+
 def run_design(args) -> int:
     import numpy as np
     import torch
@@ -406,7 +434,7 @@ def run_design(args) -> int:
     # design -> (its configuration at a size, the closest model it is measured beside)
     designs = {"tugelorn": (tugelorn_config, "qwen3"), "dufizen": (dufizen_config, "tugelorn"),
                "burolorn": (burolorn_config, "qwen3"), "gevovik": (gevovik_config, "tugelorn"),
-               "duzizen": (duzizen_config, "dufizen")}
+               "duzizen": (duzizen_config, "dufizen"), "toripel": (toripel_config, "dufizen")}
     if args.design not in designs:
         print(json.dumps({"error": f"unknown design {args.design!r}"}))
         return 2
@@ -449,10 +477,12 @@ def run_design(args) -> int:
         for b in range(B):
             eng.open_request(b)
             eng.step([StepEntry(b, rng.randint(0, V, size=ctx).tolist(), [])])
+        def ids():   # (different tokens: a design may choose experts by token id)
+            return [StepEntry(b, [int(rng.randint(0, V))], [0]) for b in range(B)]
         for _ in range(max(3, args.warmup)):
-            eng.step([StepEntry(b, [7], [0]) for b in range(B)])
+            eng.step(ids())
         l0 = kernels.counters.own + kernels.counters.library
-        ms = timed(lambda: [eng.step([StepEntry(b, [9], [0]) for b in range(B)]) for _ in range(steps)], 3)
+        ms = timed(lambda: [eng.step(ids()) for _ in range(steps)], 3)
         launches = (kernels.counters.own + kernels.counters.library - l0) // (3 * steps)
         for b in range(B):
             eng.close_request(b)
@@ -525,7 +555,7 @@ def main() -> int:
     ap.add_argument("--shape", default="8b", choices=["8b", "14b", "32b"], help="layer shape of --profile-steps")
     ap.add_argument("--workload", default="decode", choices=["decode", "mix14b", "long32b"],
                     help="decode (the default line) or one of the two other workloads of the benchmark record")
-    ap.add_argument("--design", default=None, help="tugelorn (beside Qwen3), dufizen (beside Tugelorn), burolorn (beside Qwen3), gevovik (beside Tugelorn) or duzizen (beside Dufizen): that design beside its closest model at "
+    ap.add_argument("--design", default=None, help="tugelorn (beside Qwen3), dufizen (beside Tugelorn), burolorn (beside Qwen3), gevovik (beside Tugelorn), duzizen or toripel (beside Dufizen): that design beside its closest model at "
                                                    "equal layer sizes")
     ap.add_argument("--design-sizes", default="mid,8b", help="layer sizes of --design: " + ", ".join(DESIGN_SIZES))
     ap.add_argument("--design-profile", action="store_true", help="with --design: a prompt and four eager decode steps")

@@ -154,17 +154,21 @@ struct ExpertTable {
   int* status;
 };
 
-// The expert of choice k of row t, or -1.
-__device__ __forceinline__ int table_expert(const ExpertTable& a, int t, int k) {
-  if (a.entry_of_token != nullptr && a.entry_of_token[t] < 0) return -1;
-  int id = a.ids[t];
+constexpr int kNoToken = -0x7fffffff;   // of a row that pads the step
+
+// The token of row t.
+__device__ __forceinline__ int table_token(const ExpertTable& a, int t) {
+  const int entry = a.entry_of_token != nullptr ? a.entry_of_token[t] : 0;
+  int id = a.ids[t];   // (asked for together with the entry)
   if (id < 0 && a.pending != nullptr && -1 - id < a.n_pending) id = a.pending[-1 - id];
-  const int e = id >= 0 && id < a.vocab ? a.table[(size_t)id * a.top + k] : -1;
-  if (e < 0 || e >= a.E) {
-    set_status(a.status, CCB_ST_BAD_TOKEN);
-    return -1;
-  }
-  return e;
+  return entry < 0 ? kNoToken : id;
+}
+
+// The expert of choice k of a token: -1 for a row that pads the step, -2 for a token or an expert out of range.
+__device__ __forceinline__ int table_expert(const ExpertTable& a, int id, int k) {
+  const bool in = id >= 0 && id < a.vocab;
+  const int e = in ? a.table[(size_t)id * a.top + k] : -1;
+  return e >= 0 && e < a.E ? e : (id == kNoToken ? -1 : -2);
 }
 
 // dense_w [T, E]: the weight where the table names the expert, else 0.  A thread per row and expert.
@@ -175,8 +179,12 @@ moe_table_route_kernel(const ExpertTable a, float* __restrict__ dense_w, int row
   if (i >= rows * a.E) return;
   const int t = i / a.E, e = i - t * a.E;
   float v = 0.f;
-  for (int k = 0; k < a.top; ++k)
-    if (table_expert(a, t, k) == e) v = a.weight;
+  const int id = table_token(a, t);
+  for (int k = 0; k < a.top; ++k) {
+    const int x = table_expert(a, id, k);
+    if (x == e) v = a.weight;
+    if (x == -2) set_status(a.status, CCB_ST_BAD_TOKEN);
+  }
   dense_w[i] = v;
 }
 
@@ -377,10 +385,20 @@ constexpr int kSortThreads = 1024;
 
 // idx, wts [pairs] (pairs = tokens * top).  Outputs: src_row [pairs] (token of a sorted row), row_w [pairs],
 // pair_pos [pairs] (sorted row of a pair), tile_e / tile_r0 / tile_n [max_tiles].
-// The whole block; sm: 4 E + 2 ints of shared memory.  expert_of(p), weight_of(p): of pair p (the expert negative: the
+// The whole block; sm: 4 E + 2 ints of shared memory.  Source: where a pair's expert and weight come from, the expert in
+// two steps, expert(p, first(p)), so that the loads of several pairs are in flight together (an expert out of range: the
 // pair is left out).
-template <typename ExpertOf, typename WeightOf>
-__device__ __forceinline__ void sort_pairs(ExpertOf expert_of, WeightOf weight_of, int pairs,
+struct PairLists {
+  const int* idx;
+  const float* wts;
+  __device__ __forceinline__ int first(int p) const { return idx[p]; }
+  __device__ __forceinline__ int expert(int, int e) const { return e; }
+  __device__ __forceinline__ float weight(int p) const { return wts[p]; }
+};
+
+// kBatch: pairs a thread has in flight (few pairs: one, and the code that a single block runs once stays short).
+template <int kBatch, typename Source>
+__device__ __forceinline__ void sort_pairs(const Source& from, int pairs,
                                            int top, int E, int BM, int max_tiles, int* __restrict__ src_row,
                                            float* __restrict__ row_w, int* __restrict__ pair_pos,
                                            int* __restrict__ tile_e, int* __restrict__ tile_r0,
@@ -392,9 +410,27 @@ __device__ __forceinline__ void sort_pairs(ExpertOf expert_of, WeightOf weight_o
   int* cursor = tstart + E + 1; // [E]
   for (int e = threadIdx.x; e < E; e += kSortStride) counts[e] = 0, cursor[e] = 0;
   __syncthreads();
-  for (int p = threadIdx.x; p < pairs; p += kSortStride) {
-    const int e = expert_of(p);
-    if (e >= 0 && e < E) atomicAdd(&counts[e], 1);
+  // (a pair's expert waits in pair_pos for the second pass)
+  for (int p0 = threadIdx.x; p0 < pairs; p0 += kSortStride * kBatch) {
+    int e[kBatch];
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      const int p = p0 + i * kSortStride;
+      e[i] = p < pairs ? from.first(p) : -1;
+    }
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      const int p = p0 + i * kSortStride;
+      e[i] = p < pairs ? from.expert(p, e[i]) : -1;
+    }
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      const int p = p0 + i * kSortStride;
+      if (p >= pairs) continue;
+      if (e[i] < 0 || e[i] >= E) e[i] = -1;
+      else atomicAdd(&counts[e[i]], 1);
+      pair_pos[p] = e[i];
+    }
   }
   __syncthreads();
   if (threadIdx.x == 0) {
@@ -409,13 +445,24 @@ __device__ __forceinline__ void sort_pairs(ExpertOf expert_of, WeightOf weight_o
     tstart[E] = t;
   }
   __syncthreads();
-  for (int p = threadIdx.x; p < pairs; p += kSortStride) {
-    const int e = expert_of(p);
-    if (e < 0 || e >= E) { pair_pos[p] = -1; continue; }
-    const int pos = offs[e] + atomicAdd(&cursor[e], 1);
-    src_row[pos] = p / top;
-    row_w[pos] = weight_of(p);
-    pair_pos[p] = pos;
+  for (int p0 = threadIdx.x; p0 < pairs; p0 += kSortStride * kBatch) {
+    int e[kBatch];
+    float w[kBatch];
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      const int p = p0 + i * kSortStride;
+      e[i] = p < pairs ? pair_pos[p] : -1;   // (written by this thread)
+      w[i] = e[i] >= 0 ? from.weight(p) : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      const int p = p0 + i * kSortStride;
+      if (e[i] < 0) continue;
+      const int pos = offs[e[i]] + atomicAdd(&cursor[e[i]], 1);
+      src_row[pos] = p / top;
+      row_w[pos] = w[i];
+      pair_pos[p] = pos;
+    }
   }
   for (int p = offs[E] + threadIdx.x; p < pairs; p += kSortStride) {   // (places of pairs that were left out)
     src_row[p] = 0;
@@ -440,26 +487,38 @@ __device__ __forceinline__ void sort_pairs(ExpertOf expert_of, WeightOf weight_o
   }
 }
 
+constexpr int kSortBatch = 8;   // from more pairs than threads on
+
+template <int kBatch>
 __global__ void __launch_bounds__(kSortThreads)
 moe_sort_kernel(const int* __restrict__ idx, const float* __restrict__ wts, int pairs, int top, int E, int BM,
                 int max_tiles, int* __restrict__ src_row, float* __restrict__ row_w, int* __restrict__ pair_pos,
                 int* __restrict__ tile_e, int* __restrict__ tile_r0, int* __restrict__ tile_n) {
   ccb::pdl_begin();
   extern __shared__ int sm[];
-  sort_pairs([&](int p) { return idx[p]; }, [&](int p) { return wts[p]; }, pairs, top, E, BM, max_tiles, src_row, row_w,
-             pair_pos, tile_e, tile_r0, tile_n, sm);
+  sort_pairs<kBatch>(PairLists{idx, wts}, pairs, top, E, BM, max_tiles, src_row, row_w, pair_pos, tile_e, tile_r0, tile_n, sm);
 }
 
 // The sort with the experts read from a table as it goes: there are no idx and wts.
+struct PairTable {
+  const ExpertTable& a;
+  __device__ __forceinline__ int first(int p) const { return table_token(a, p / a.top); }
+  __device__ __forceinline__ int expert(int p, int id) const {
+    const int e = table_expert(a, id, p % a.top);
+    if (e == -2) set_status(a.status, CCB_ST_BAD_TOKEN);
+    return e;
+  }
+  __device__ __forceinline__ float weight(int) const { return a.weight; }
+};
+
+template <int kBatch>
 __global__ void __launch_bounds__(kSortThreads)
 moe_table_sort_kernel(const ExpertTable a, int pairs, int BM, int max_tiles, int* __restrict__ src_row,
                       float* __restrict__ row_w, int* __restrict__ pair_pos, int* __restrict__ tile_e,
                       int* __restrict__ tile_r0, int* __restrict__ tile_n) {
   ccb::pdl_begin();
   extern __shared__ int sm[];
-  sort_pairs([&](int p) { const int t = p / a.top; return table_expert(a, t, p - t * a.top); },
-             [&](int) { return a.weight; }, pairs, a.top, a.E, BM, max_tiles, src_row, row_w, pair_pos, tile_e, tile_r0,
-             tile_n, sm);
+  sort_pairs<kBatch>(PairTable{a}, pairs, a.top, a.E, BM, max_tiles, src_row, row_w, pair_pos, tile_e, tile_r0, tile_n, sm);
 }
 
 // Steps of few tokens: the router and the sort in one block, a warp a token (up to 32 tokens).
@@ -479,8 +538,7 @@ moe_route_sort_kernel(const float* __restrict__ logits, int ldl, const float* __
                 scratch + (size_t)warp * (2 * E + groups), lane, rule);
   __threadfence_block();
   __syncthreads();   // the choices are written: the same block sorts them
-  sort_pairs([&](int p) { return idx[p]; }, [&](int p) { return wts[p]; }, rows * top, top, E, BM, max_tiles, src_row, row_w,
-             pair_pos, tile_e, tile_r0, tile_n, sm);
+  sort_pairs<1>(PairLists{idx, wts}, rows * top, top, E, BM, max_tiles, src_row, row_w, pair_pos, tile_e, tile_r0, tile_n, sm);
 }
 
 __device__ __forceinline__ uint4 ld16_or_zero(const __nv_bfloat16* p, bool ok) {
@@ -705,8 +763,9 @@ CCB_API int ccb_moe_sort(const int* idx, const float* wts, int pairs, int top, i
   if (E <= 0 || top <= 0 || BM <= 0 || max_tiles < min(pairs, (pairs + BM - 1) / BM + E)) return CCB_REFUSE_SIZE;
   const size_t smem = (size_t)(4 * E + 2) * sizeof(int);
   if (smem > 96 * 1024) return CCB_REFUSE_SIZE;
-  cudaFuncSetAttribute(moe_sort_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  ccb_launch(moe_sort_kernel, dim3(1), dim3(kSortThreads), smem, stream, idx, wts, pairs, top, E, BM, max_tiles,
+  const auto kernel = pairs > kSortThreads ? moe_sort_kernel<kSortBatch> : moe_sort_kernel<1>;
+  cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  ccb_launch(kernel, dim3(1), dim3(kSortThreads), smem, stream, idx, wts, pairs, top, E, BM, max_tiles,
              src_row, row_w, pair_pos, tile_e, tile_r0, tile_n);
   return ccb_launch_status();
 }
@@ -734,8 +793,9 @@ CCB_API int ccb_moe_table_sort(const int* table, const int* ids, const int* entr
   const ExpertTable a{table, ids, entry_of_token, pending, top, E, vocab, n_pending, weight, status};
   const size_t smem = (size_t)(4 * E + 2) * sizeof(int);
   if (smem > 96 * 1024) return CCB_REFUSE_SIZE;
-  cudaFuncSetAttribute(moe_table_sort_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  ccb_launch(moe_table_sort_kernel, dim3(1), dim3(kSortThreads), smem, stream, a, pairs, BM, max_tiles, src_row, row_w,
+  const auto kernel = pairs > kSortThreads ? moe_table_sort_kernel<kSortBatch> : moe_table_sort_kernel<1>;
+  cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  ccb_launch(kernel, dim3(1), dim3(kSortThreads), smem, stream, a, pairs, BM, max_tiles, src_row, row_w,
              pair_pos, tile_e, tile_r0, tile_n);
   return ccb_launch_status();
 }

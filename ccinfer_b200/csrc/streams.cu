@@ -14,17 +14,20 @@
 // `table`: the copies come straight from the embedding: x = table[ids[t]] * scale is written to x_out ([T, D]) and y
 // is the first sublayer's norm.
 //
-//   streams_vec   D a multiple of 4 up to 8,192 with aligned rows: 16-byte accesses, u stays in registers
+//   streams_vec   D a multiple of 4 up to 8,192 with aligned rows: 16-byte accesses, u stays in registers.  Few rows: a
+//                 cluster of up to eight blocks shares a row (the copies of one row alone are tens of kilobytes), and
+//                 their sums of squares meet through distributed shared memory
 //   streams_row   any D whose row fits shared memory
 //
 // Everything is float but d, y and the table.
-#include "common.cuh"
+#include "cluster_common.cuh"
 
 using namespace ccb;
 
 namespace {
 
 constexpr int kMaxStreams = 16;
+constexpr int kClusterMaxRows = 64;   // up to this many rows a cluster shares each
 
 struct StreamsArgs {
   const float* x;          // [rows, S, D], or [rows, D] with `shared`
@@ -77,15 +80,25 @@ __device__ __forceinline__ int token_of(const StreamsArgs& a, int t) {
   return id >= 0 && id < a.vocab ? id : -1;
 }
 
-// SS: copies (0: a.S of them, a loop).  kAhead: the norm's weight is asked for before the row.
-template <typename T, int SS, int NV, int kThreads, bool kAhead>
+// SS: copies (0: a.S of them, a loop).  kAhead: the norm's weight is asked for before the row.  kCluster: the blocks of a
+// cluster share a row, side by side (NV 1).
+template <typename T, int SS, int NV, int kThreads, bool kAhead, bool kCluster>
 __global__ void __launch_bounds__(kThreads)
 streams_vec_kernel(T* __restrict__ y, const StreamsArgs a) {
   constexpr int SM = SS > 0 ? SS : kMaxStreams;
   const int S = SS > 0 ? SS : a.S;
   __shared__ float red[32];
+  __shared__ float slots[kMaxClusterBlocks];
   __shared__ float coef[kMaxStreams * kMaxStreams + 2 * kMaxStreams];   // mix, out, in
-  const int r = blockIdx.x;
+  static_assert(!kCluster || NV == 1, "a block of a cluster holds one run of columns");
+  int r = blockIdx.x, base = 0;
+  if constexpr (kCluster) {
+    cluster_arrive();
+    const int n = (int)cooperative_groups::this_cluster().num_blocks();
+    r = blockIdx.x / n;
+    base = (blockIdx.x % n) * kThreads;
+  }
+  const int first = base + threadIdx.x;   // this thread's vectors of four columns: first, first + kThreads, ...
   const int D = a.D, nvec = D >> 2;
   float* mix_s = coef;
   float* out_s = coef + kMaxStreams * kMaxStreams;
@@ -100,7 +113,7 @@ streams_vec_kernel(T* __restrict__ y, const StreamsArgs a) {
   if (kAhead && y != nullptr) {
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
-      const int i = threadIdx.x + j * kThreads;
+      const int i = first + j * kThreads;
       if (i < nvec) w[j] = V4<float>::load(a.w + 4 * i);
     }
   }
@@ -108,13 +121,20 @@ streams_vec_kernel(T* __restrict__ y, const StreamsArgs a) {
   __syncthreads();
   const int src = a.row_idx ? a.row_idx[r] : r;
   T* yr = y ? y + (size_t)r * D : nullptr;
-  if (src < 0 || src >= a.n_src_rows) {
+  const bool bad = src < 0 || src >= a.n_src_rows;
+  if (bad) {
     if (threadIdx.x == 0) set_status(a.status, CCB_ST_BAD_ROW);
     if (yr)
-      for (int i = threadIdx.x; i < nvec; i += kThreads) V4<T>::store(yr + 4 * i, make_float4(0.f, 0.f, 0.f, 0.f));
-    return;
+      for (int i = first; i < nvec; i += (kCluster ? nvec : kThreads))
+        V4<T>::store(yr + 4 * i, make_float4(0.f, 0.f, 0.f, 0.f));
+    if constexpr (!kCluster) return;
   }
   float4 u[NV];
+#pragma unroll
+  for (int j = 0; j < NV; ++j) u[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (kCluster && bad) {
+    // (the blocks of a cluster meet below, whatever their row)
+  } else
   if (a.table != nullptr) {
     const int id = token_of(a, src);
     if (id < 0 && threadIdx.x == 0) set_status(a.status, CCB_ST_BAD_TOKEN);
@@ -123,7 +143,7 @@ streams_vec_kernel(T* __restrict__ y, const StreamsArgs a) {
     const T* er = static_cast<const T*>(a.table) + (size_t)(id < 0 ? 0 : id) * D;
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
-      const int i = threadIdx.x + j * kThreads;
+      const int i = first + j * kThreads;
       if (i < nvec) {
         float4 v = V4<T>::load(er + 4 * i);
         const float f = id < 0 ? 0.f : a.scale;
@@ -139,7 +159,7 @@ streams_vec_kernel(T* __restrict__ y, const StreamsArgs a) {
     const int* pp = a.pair_rows ? a.pair_pos + (size_t)src * a.top : nullptr;
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
-      const int i = threadIdx.x + j * kThreads;
+      const int i = first + j * kThreads;
       if (i >= nvec) continue;
       float4 x[SM], d = make_float4(0.f, 0.f, 0.f, 0.f);
       if (a.shared) {
@@ -153,6 +173,7 @@ streams_vec_kernel(T* __restrict__ y, const StreamsArgs a) {
       }
       if (dr) d = V4<T>::load(dr + 4 * i);
       if (pp) {
+#pragma unroll 4
         for (int k = 0; k < a.top; ++k) {
           const int p = pp[k];
           if (p >= 0 && p < a.n_pair_rows) axpy4(d, 1.f, V4<float>::load(a.pair_rows + (size_t)p * D + 4 * i));
@@ -179,17 +200,23 @@ streams_vec_kernel(T* __restrict__ y, const StreamsArgs a) {
       u[j] = uj;
     }
   }
-  if (yr == nullptr) return;
+  if constexpr (!kCluster) {
+    if (yr == nullptr) return;
+  }
   float ss = 0.f;
 #pragma unroll
   for (int j = 0; j < NV; ++j)
-    if (threadIdx.x + j * kThreads < nvec)
+    if (first + j * kThreads < nvec)
       ss += (u[j].x * u[j].x + u[j].y * u[j].y) + (u[j].z * u[j].z + u[j].w * u[j].w);
   ss = block_sum<kThreads>(ss, red);
+  if constexpr (kCluster) {
+    ss = cluster_sum(ss, slots);
+    if (yr == nullptr || bad) return;
+  }
   const float inv = 1.0f / sqrtf(ss / (float)D + a.eps);
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
-    const int i = threadIdx.x + j * kThreads;
+    const int i = first + j * kThreads;
     if (i >= nvec) continue;
     const float4 wj = kAhead ? w[j] : V4<float>::load(a.w + 4 * i);
     V4<T>::store(yr + 4 * i, make_float4(u[j].x * inv * wj.x, u[j].y * inv * wj.y, u[j].z * inv * wj.z,
@@ -255,8 +282,16 @@ __global__ void __launch_bounds__(kRowThreads) streams_row_kernel(T* __restrict_
 template <typename T, int SS>
 void launch_vec(void* y, const StreamsArgs& a, int rows, cudaStream_t stream) {
 #define CCB_STREAMS(NV, TH, AH)                                                                                       \
-  ccb_launch_ex(AH, streams_vec_kernel<T, SS, NV, TH, AH>, dim3(rows), dim3(TH), 0, stream, (T*)y, a)
+  ccb_launch_ex(AH, streams_vec_kernel<T, SS, NV, TH, AH, false>, dim3(rows), dim3(TH), 0, stream, (T*)y, a)
   const int D = a.D;
+  if (D > 512 && rows <= kClusterMaxRows) {   // 512 or 1,024 columns a block
+    const int threads = D <= 4096 ? 128 : 256, n = (D / 4 + threads - 1) / threads;
+    if (threads == 128)
+      ccb_launch_cluster(true, n, streams_vec_kernel<T, SS, 1, 128, true, true>, dim3(rows * n), dim3(128), 0, stream, (T*)y, a);
+    else
+      ccb_launch_cluster(true, n, streams_vec_kernel<T, SS, 1, 256, true, true>, dim3(rows * n), dim3(256), 0, stream, (T*)y, a);
+    return;
+  }
   if (rows <= 148) {
     if (D <= 512) CCB_STREAMS(1, 128, true);
     else if (D <= 1024) CCB_STREAMS(1, 256, true);

@@ -381,6 +381,12 @@ class GroupedQueryAttention(Mixer):
                 and step.n_single == step.n_entries == step.n_tokens
                 and step.n_tokens <= self.FUSED_DECODE_MAX_ROWS)
 
+    def _q_rows(self):
+        """Buffer for the queries where they leave the projection's rows (layers of other sizes have buffers of their own:
+        a step of single tokens may not use it, and it must not grow once graphs hold the pool's addresses)."""
+        rt = self.rt
+        return rt.scratch.get(f"attn_q:{self.nq * self.hd}", (rt.max_tokens, self.nq, self.hd), rt.dtype)
+
     def _convolve(self, qkv, step, state, T):
         """The rows of q | k | v after the short convolution (state: the last taps - 1 rows of each request) and
         the mixing of the values with the first such layer's."""
@@ -414,7 +420,7 @@ class GroupedQueryAttention(Mixer):
             qkv = self._convolve(qkv, step, state, T)
         o = rt.scratch.get("attn_o", (rt.max_tokens, self.nq, self.hd), rt.dtype)[:T]
         if self.keys_as_values:
-            q = rt.scratch.get("attn_q", (rt.max_tokens, self.nq, self.hd), rt.dtype)[:T]
+            q = self._q_rows()[:T]
             taps = max(self.taps, 1)
             kernels.qk_rows(qkv, q, cache.k, cache.v, self.conv_w, taps, state, self.q_norm_w, self.k_norm_w,
                             self.norm_eps if self.norm_eps is not None else 1.0, self.qk_dim,
@@ -439,7 +445,7 @@ class GroupedQueryAttention(Mixer):
                 bias=self.bias, q_temperature=self.position.query_temperature(), chunk=self.chunk, sink=self.sink,
                 gate=gate, keep=self.keep_first)
         else:
-            q = rt.scratch.get("attn_q", (rt.max_tokens, self.nq, self.hd), rt.dtype)[:T]
+            q = self._q_rows()[:T]
             args = (qkv, q, cache.k if self.own_kv else None, cache.v if self.own_kv else None, step.positions,
                     g.slot_map if self.own_kv else None, self.position.rotary_table(), self.q_norm_w, self.k_norm_w,
                     self.norm_eps if self.norm_eps is not None else 1.0, self.nq, nkv_w, self.hd, g.page_size)

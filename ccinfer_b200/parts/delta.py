@@ -225,12 +225,14 @@ class HeadGatedDelta(Mixer):
             kernels.delta_head_step(self.rule, proj, ring, S, self.norm_w, self.eps, step.positions, step.cu_q,
                                     step.state_slot, y, n1)
         if many > 0:
-            qn = rt.scratch.get("delta_q", (rt.max_tokens, G, dk), f32)[:T]
-            kn = rt.scratch.get("delta_k", (rt.max_tokens, G, dk), f32)[:T]
-            vv = rt.scratch.get("delta_v", (rt.max_tokens, H, dv), f32)[:T]
-            gg = rt.scratch.get("delta_decay", (rt.max_tokens, H), f32)[:T]
-            bb = rt.scratch.get("delta_beta", (rt.max_tokens, H), f32)[:T]
-            o = rt.scratch.get("delta_o", (rt.max_tokens, H, dv), f32)[:T]
+            # (layers of other sizes have buffers of their own: what only portions use must not grow once graphs hold the
+            # pool's addresses)
+            qn = rt.scratch.get(f"delta_q:{G * dk}", (rt.max_tokens, G, dk), f32)[:T]
+            kn = rt.scratch.get(f"delta_k:{G * dk}", (rt.max_tokens, G, dk), f32)[:T]
+            vv = rt.scratch.get(f"delta_v:{H * dv}", (rt.max_tokens, H, dv), f32)[:T]
+            gg = rt.scratch.get(f"delta_decay:{H}", (rt.max_tokens, H), f32)[:T]
+            bb = rt.scratch.get(f"delta_beta:{H}", (rt.max_tokens, H), f32)[:T]
+            o = rt.scratch.get(f"delta_o:{H * dv}", (rt.max_tokens, H, dv), f32)[:T]
             kernels.delta_head_prepare(self.rule, proj, ring, step.positions, step.entry_of_token, step.cu_q,
                                        step.state_slot, qn, kn, vv, gg, bb, n1, T - n1)
             kernels.conv_ring_write(self.rule, proj, ring, step.positions, step.cu_q, step.state_slot, n1, many)
