@@ -322,10 +322,10 @@ delta_head_prepare_kernel(const T* __restrict__ proj, const T* __restrict__ ring
 
 // The same with four channels a lane and kRun neighbouring rows a warp: the taps' weights are loaded once for all of them,
 // a row once for all the taps it meets, and all are in flight together.  dk, dv multiples of 4, dk <= 128 X, TAPS taps.
-constexpr int kRun = 8;
+constexpr int kRun = 4;
 
 template <typename T, int TAPS, int X>
-__global__ void __launch_bounds__(kPrepWarps * 32, sizeof(T) == 2 && X == 1 ? 6 : 3)   // (latency: warps count)
+__global__ void __launch_bounds__(kPrepWarps * 32, sizeof(T) == 2 && X == 1 ? 7 : 3)   // (latency: warps count)
 delta_head_prepare_run_kernel(const T* __restrict__ proj, const T* __restrict__ ring, float* __restrict__ qn,
                               float* __restrict__ kn, float* __restrict__ vv, float* __restrict__ gg,
                               float* __restrict__ bb, int row0, int row_end, const HeadDelta a) {
