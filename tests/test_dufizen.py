@@ -410,7 +410,7 @@ def test_replay_with_the_sparse_experts(models, name, dtype, monkeypatch):
     monkeypatch.setattr(MixtureOfExperts, "SPARSE_MIN_WEIGHTS", 0)
     calls = []
     inner = MixtureOfExperts._forward_sparse
-    monkeypatch.setattr(MixtureOfExperts, "_forward_sparse", lambda self, x, T: (calls.append(T), inner(self, x, T))[1])
+    monkeypatch.setattr(MixtureOfExperts, "_forward_sparse", lambda self, x, T, step: (calls.append(T), inner(self, x, T, step))[1])
     d, cfg, w, reqs, ref, page = models[name, dtype]
     for steps, graphs in ((helpers.trace_whole(reqs), False), (helpers.trace_mixed(reqs, max_live=4, seed=7), True)):
         pool = helpers.max_live_tokens(steps, round_to=max(64, page))
