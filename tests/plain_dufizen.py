@@ -102,6 +102,15 @@ def latent_attention_mixer(h, W, p, m, eps, use_sink=True):
     return o.reshape(T, H * dv) @ W[p + "o"].T
 
 
+choice_gaps = None   # a list: ``route`` adds every token's distance between what is chosen and what just is not
+
+
+def _note_gap(values, keep):
+    v = values.sort(-1, descending=True).values
+    if choice_gaps is not None and keep < v.shape[-1]:
+        choice_gaps.append(v[:, keep - 1] - v[:, keep])
+
+
 def route(z, correction, r):
     """Router logits z [T, E] -> (indices [T, top], weights [T, top])."""
     E, top = r["experts"], r["top"]
@@ -109,9 +118,11 @@ def route(z, correction, r):
     choice = s + correction
     if r.get("groups") is not None:
         G, keep = r["groups"]["count"], r["groups"]["keep"]
+        _note_gap(choice.view(-1, G, E // G).max(-1).values, keep)
         best = choice.view(-1, G, E // G).max(-1).values.topk(keep, -1).indices
         ok = torch.zeros(z.shape[0], G, dtype=torch.bool).scatter_(1, best, True)
         choice = choice.masked_fill(~ok[:, :, None].expand(-1, G, E // G).reshape(-1, E), -math.inf)
+    _note_gap(choice, top)
     idx = choice.topk(top, -1).indices
     return idx, s.gather(1, idx)
 
